@@ -16,7 +16,8 @@
 //                          forget gate, state in fp32 carried in device memory, per-head RMS norm of o fused
 //   dual_norm_hc_kernel    y = 1/2 (rmsnorm(a) wa + rmsnorm(b) wb) -> layer scale -> hyper-connection write
 //   group_norm_residual_kernel  x + grouped RMS norm of a sublayer's output (weighted sum of expert rows first), depth-weighted average
-//   qkv_post_kernel        bias, rotary positions, weightless RMS norms of q / k / v heads, K/V cache write (kept first slots + ring)
+//   qkv_post_kernel        bias, rotary positions, RMS norms of q / k / v heads, query temperature, K/V cache write (kept first slots + ring)
+//   layer_norm_kernel      (x - mean) / sqrt(variance + eps) * w + b
 //
 // The kernels have internal linkage: every translation unit that includes this header (a model family, the op-level entry points
 // of mix_ops.cu) gets its own copies.
@@ -82,13 +83,16 @@ struct SeqStep {
 };
 
 // ---- embedding -> streams -------------------------------------------------------------------------------------------------
+// positions: (max positions, width) learned rows, the one of the token's position in its sequence is added (unscaled); NULL: none
 template <typename WT>
 __global__ void embed_streams_kernel(const WT* __restrict__ table, const int* __restrict__ tokens, int width, int S, size_t stream_stride,
-                                     float* __restrict__ xs, float scale = 1.f) {
+                                     float* __restrict__ xs, float scale = 1.f, const WT* __restrict__ positions = nullptr, const SeqStep* step = nullptr) {
 	const int t = blockIdx.x;
 	const WT* row = table + (size_t) tokens[t] * width;
+	const WT* prow = positions ? positions + (size_t) (step->pos0 + t) * width : nullptr;
 	for (int c = threadIdx.x; c < width; c += blockDim.x) {
-		const float v = ldf(row + c) * scale; // scale 1: the row as it is
+		float v = ldf(row + c) * scale; // scale 1: the row as it is
+		if (prow) v += ldf(prow + c);
 		for (int s = 0; s < S; s++) xs[(size_t) s * stream_stride + (size_t) t * width + c] = v;
 	}
 }
@@ -204,6 +208,48 @@ __global__ void hc_norm_kernel(const float* __restrict__ xs, int S, size_t strea
 	}
 }
 
+// ---- layer norm ------------------------------------------------------------------------------------------------------------------
+// h[t] = (x[t] - mean) / sqrt(mean of the squared deviations + eps) * w + b (b NULL: no bias).  One CTA per row; the row stays in shared memory
+// between the two sums, so the deviations are taken from the finished mean.  Loads four columns per thread ahead, as hc_norm_kernel.
+static __global__ void layer_norm_kernel(const float* __restrict__ x, int ldx, const float* __restrict__ w, const float* __restrict__ b, float eps, int width,
+                                         float* __restrict__ h) {
+	extern __shared__ float sm[];
+	float* u = sm;            // width
+	float* red = sm + width;  // 33
+	const int t = blockIdx.x, tid = threadIdx.x, nth = blockDim.x;
+	const float* row = x + (size_t) t * ldx;
+	float tot = 0.f;
+	for (int c0 = tid; c0 < width; c0 += 4 * nth) {
+		float v[4];
+#pragma unroll
+		for (int k = 0; k < 4; k++) v[k] = c0 + k * nth < width ? row[c0 + k * nth] : 0.f;
+#pragma unroll
+		for (int k = 0; k < 4; k++) {
+			if (c0 + k * nth < width) u[c0 + k * nth] = v[k];
+			tot += v[k];
+		}
+	}
+	const float mean = block_sum(tot, red) / (float) width;
+	float ss = 0.f;
+	for (int c = tid; c < width; c += nth) { // columns this thread wrote
+		const float dv = u[c] - mean;
+		ss = fmaf(dv, dv, ss);
+	}
+	const float r = 1.f / sqrtf(block_sum(ss, red) / (float) width + eps);
+	for (int c0 = tid; c0 < width; c0 += 4 * nth) {
+		float wv[4], bv[4];
+#pragma unroll
+		for (int k = 0; k < 4; k++) {
+			const bool in = c0 + k * nth < width;
+			wv[k] = in ? w[c0 + k * nth] : 0.f;
+			bv[k] = in && b ? b[c0 + k * nth] : 0.f;
+		}
+#pragma unroll
+		for (int k = 0; k < 4; k++)
+			if (c0 + k * nth < width) h[(size_t) t * width + c0 + k * nth] = fmaf((u[c0 + k * nth] - mean) * r, wv[k], bv[k]);
+	}
+}
+
 // ---- fused epilogues of the row products -------------------------------------------------------------------------------------
 enum { EPI_STORE = 0, EPI_SPLIT_KV = 1, EPI_GLU = 2, EPI_HC = 3, EPI_ACT = 4 };
 enum { GLU_CLAMPED = 0, GLU_SILU = 1, GLU_GELU_TANH = 2 };
@@ -217,6 +263,10 @@ struct RowsEpi {
 	float cap = 0.f;
 	const float* mul = nullptr;
 	int ldm = 0, mul_act = ACT_SIGMOID;
+	// STORE, last: v <- v + add[row * lda + col] when add is set (the other half of a product over two operands side by side; may be `out`
+	// itself: each value is read by the thread that writes it).  Not for batched products
+	const float* add = nullptr;
+	int lda = 0;
 	// ACT: v <- act(v + bias[col]), no gate.  ACT_SIGMOID_POW: sigmoid(.)^act_pow, as exp(act_pow * log sigmoid(.)) (a decay in (0, 1) whose
 	// logarithm stays exact where the sigmoid itself would leave the fp32 range)
 	int act = ACT_NONE;
@@ -292,6 +342,7 @@ __device__ __forceinline__ void epi_apply(const RowsEpi& e, int row, int col, in
 		case EPI_STORE:
 			if (e.cap > 0.f) v = e.cap * tanhf(v / e.cap);
 			if (e.mul) v *= act_apply(e.mul_act, e.mul[(size_t) row * e.ldm + col]);
+			if (e.add) v += e.add[(size_t) row * e.lda + col];
 			e.out[(size_t) row * e.ldo + col] = v;
 			break;
 		case EPI_ACT: e.out[(size_t) row * e.ldo + col] = act_apply(e.act, e.bias ? v + e.bias[col] : v, e.act_pow); break;
@@ -479,6 +530,7 @@ struct SwaArgs {
 	const float* q;    // (T, ldq): head h at columns q_off + h * d
 	const float* gate; // (T, ldg): pre-sigmoid gate of the concatenated heads at columns g_off + ...; NULL: no gate
 	int ldq, q_off, ldg, g_off;
+	int gate_per_head; // 1: one gate value per head, at column g_off + h
 	const void* kc;    // ring (ring, G * d)
 	const void* vc;    // ring (ring, G * dv)
 	int ldk, ldv;      // elements between the rows of two slots; 0: G * d and G * dv.  A cache whose rows hold more than the keys (values that
@@ -492,6 +544,7 @@ struct SwaArgs {
 	float softcap;     // 0: none
 	const float* r1;   // distance bias r1[h] * log1p(r2[h] * (i - j)) taken off the score; NULL: none
 	const float* r2;
+	const float* slope; // (H) linear distance bias slope[h] * (i - j) taken off the score; NULL: none
 	const float* talk; // (H, H) score_h <- sum_g talk[h, g] score_g; NULL: none
 	const float* sink; // (H) the softmax's denominator also holds exp(sink[h]): a key of no position and no value that is not scaled; NULL: none
 	float out_scale;   // multiplies the result (0: 1)
@@ -545,6 +598,11 @@ __device__ __forceinline__ float swa_finish(const SwaArgs& a, int h, float num, 
 	return a.out_scale != 0.f ? o * a.out_scale : o;
 }
 
+// sigmoid of the gate of head h, value column c of row t
+__device__ __forceinline__ float swa_gate(const SwaArgs& a, int t, int h, int c) {
+	return sigmoidf_(a.gate[(size_t) t * a.ldg + a.g_off + (a.gate_per_head ? h : h * a.dv + c)]);
+}
+
 // joins the key splits of rows [t_first, t_first + rows): out = (sum_s e^{m_s - m} O_s) / (sum_s e^{m_s - m} l_s), then the gate
 __device__ __forceinline__ void swa_merge_one(const SwaArgs& a, int t, int hc) {
 	const int H = a.H, dv = a.dv, ns = a.n_splits, h = hc / dv;
@@ -577,7 +635,7 @@ __device__ __forceinline__ void swa_merge_one(const SwaArgs& a, int t, int hc) {
 			}
 	}
 	float o = swa_finish(a, h, num, den, m);
-	if (a.gate) o *= sigmoidf_(a.gate[(size_t) t * a.ldg + a.g_off + hc]);
+	if (a.gate) o *= swa_gate(a, t, h, hc % dv);
 	a.out[(size_t) t * (a.ldo ? a.ldo : H * dv) + hc] = o;
 }
 __device__ __forceinline__ void swa_merge_rows(const SwaArgs& a, int t_first, int rows, int tid, int nth) {
@@ -729,6 +787,7 @@ __global__ void __launch_bounds__(256) swa_attn_kernel(SwaArgs a) {
 							sv = mine * a.scale;
 							if (a.softcap > 0.f) sv = a.softcap * tanhf(sv / a.softcap);
 							if (a.r1) sv -= a.r1[h] * log1pf(a.r2[h] * (float) (i - j));
+							if (a.slope) sv -= a.slope[h] * (float) (i - j);
 						}
 						sc[h * SWA_KB + jj] = sv;
 					}
@@ -793,7 +852,7 @@ __global__ void __launch_bounds__(256) swa_attn_kernel(SwaArgs a) {
 	if (a.n_splits == 1) {
 		for (int x = tid; x < H * dv; x += nth) {
 			float o = swa_finish(a, x / dv, O[x], lrun[x / dv], mrun[x / dv]);
-			if (a.gate) o *= sigmoidf_(a.gate[(size_t) t * a.ldg + a.g_off + x]);
+			if (a.gate) o *= swa_gate(a, t, x / dv, x % dv);
 			a.out[(size_t) t * (a.ldo ? a.ldo : H * dv) + x] = o;
 		}
 	} else {
@@ -915,6 +974,7 @@ __device__ __forceinline__ void swa_qk_tiles(const SwaArgs& a, const float* Qs, 
 					s = acc[i][u] * a.scale;
 					if (a.softcap > 0.f) s = a.softcap * tanhf(s / a.softcap);
 					if (a.r1) s -= a.r1[h] * log1pf(a.r2[h] * (float) max(i_lo + q - j, 0));
+					if (a.slope) s -= a.slope[h] * (float) max(i_lo + q - j, 0);
 				}
 				o4[i] = s;
 			}
@@ -1083,7 +1143,7 @@ __global__ void __launch_bounds__(256) swa_tile_kernel(SwaArgs a) {
 		const float acc = O[(size_t) row * dvp + c];
 		if (a.n_splits == 1) {
 			float o = swa_finish(a, h, acc, lrun[row], mrun[row]);
-			if (a.gate) o *= sigmoidf_(a.gate[(size_t) t * a.ldg + a.g_off + h * dv + c]);
+			if (a.gate) o *= swa_gate(a, t, h, c);
 			a.out[(size_t) t * (a.ldo ? a.ldo : H * dv) + h * dv + c] = o;
 		} else a.part_o[((size_t) t * a.n_splits + sp) * (H * dv) + h * dv + c] = acc;
 	}
@@ -1699,7 +1759,8 @@ static inline int launch_group_norm(const GroupNormArgs& a, int rows, cudaStream
 // One warp per head of a token.  Query heads are rewritten in place; key and value heads go to the cache slot of the token's position
 // (SwaKeys layout: the first keep_first positions in slots of their own, the rest in a ring).  Rotation: the first 2 * rot_half
 // dimensions of a query / key head, dimension i paired with i + rot_half, angle = position * freq[i] in fp32 (sincosf).  The norms
-// (x / sqrt(mean(x^2) + eps) over the head, no weight) come after the rotation; each is optional.
+// (x / sqrt(mean(x^2) + eps) over the head; q_norm_w / k_norm_w: a weight over the head's entries, shared by all heads) come after the
+// rotation; each is optional.  Last, a query at position p is multiplied by 1 + temp_coef * ln(floor((p + 1) / temp_every) + 1) when temp_every > 0.
 struct QkvPostArgs {
 	float* proj; // (T, ld)
 	int ld, q_off, k_off, v_off;
@@ -1709,6 +1770,9 @@ struct QkvPostArgs {
 	int rot_half;
 	float rot_mag;             // multiplies cos and sin of every turn (a rescaled rotation changes the length of what it turns); 0: 1
 	int norm_qk, norm_v;
+	const float *q_norm_w, *k_norm_w; // (d) or NULL (weight 1)
+	int temp_every;
+	float temp_coef;
 	float eps;
 	void *kc, *vc;
 	int cache_f32, keep_first, ring;
@@ -1748,7 +1812,14 @@ static __global__ void qkv_post_kernel(QkvPostArgs a) {
 		ss = warp_sum(ss);
 		rs = 1.f / sqrtf(ss / (float) n + a.eps);
 	}
+	if (kind != 2) {
+		const float* nw = kind == 0 ? a.q_norm_w : a.k_norm_w;
+		if (nw)
+			for (int c = lane; c < n; c += 32) x[c] = x[c] * rs * nw[c]; // a lane's own entries
+		if (nw) rs = 1.f;
+	}
 	if (kind == 0) {
+		if (a.temp_every > 0) rs *= fmaf(a.temp_coef, logf((float) ((pos + 1) / a.temp_every) + 1.f), 1.f);
 		for (int c = lane; c < n; c += 32) src[c] = x[c] * rs;
 		return;
 	}
@@ -1795,6 +1866,19 @@ static inline int launch_hc_norm(const float* xs, int S, size_t stream_stride, c
 	return launch_check("hc_norm");
 }
 
+static inline int layer_norm_prepare(int width) {
+	static bool raised = false;
+	if ((size_t) (width + 33) * 4 > 48 * 1024 && !raised) {
+		XALM_CUDA_CHECK(cudaFuncSetAttribute(layer_norm_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024));
+		raised = true;
+	}
+	return XALM_OK;
+}
+static inline int launch_layer_norm(const float* x, int ldx, const float* w, const float* b, float eps, int width, float* h, int rows, cudaStream_t s) {
+	layer_norm_kernel<<<rows, norm_threads(width), (size_t) (width + 33) * 4, s>>>(x, ldx, w, b, eps, width, h);
+	return launch_check("layer_norm");
+}
+
 // widths whose combined row fits the default 48 KB of dynamic shared memory can carry the next sublayer's read
 static inline bool dual_norm_can_carry(int width) { return (size_t) (width + 33) * 4 <= 48 * 1024; }
 static inline int launch_dual_norm_hc(const float* A, const float* B, const float* wa, const float* wb, float eps, int width, const RowsEpi& e, int rows,
@@ -1838,8 +1922,10 @@ static inline int launch_swa(SwaArgs a, int rows, bool cache_f32, cudaStream_t s
 				b.H = Hc;
 				b.ldo = a.H * a.dv;
 				b.q_off = a.q_off + z * Hc * a.d;
-				b.g_off = a.g_off + z * Hc * a.dv;
+				b.g_off = a.g_off + z * Hc * (a.gate_per_head ? 1 : a.dv);
 				if (a.sink) b.sink = a.sink + (size_t) z * Hc;
+				if (a.r1) { b.r1 = a.r1 + (size_t) z * Hc; b.r2 = a.r2 + (size_t) z * Hc; }
+				if (a.slope) b.slope = a.slope + (size_t) z * Hc;
 				b.out = a.out + (size_t) z * Hc * a.dv;
 				if (a.part_o) b.part_o = a.part_o + (size_t) z * cap * Hc * a.dv;
 				if (a.part_ml) b.part_ml = a.part_ml + (size_t) z * cap * Hc * 2;

@@ -3,9 +3,12 @@
 //   moe_router_kernel   per token: logits z = W_router h in fp32, scores s = sigmoid(z) or softmax(z) over all experts; optionally the
 //                       experts form n_groups equal groups of neighbours, a group scores the sum of its two largest s or its largest s, and
 //                       only experts of the keep_groups best groups can be chosen; the `top` largest s among those are chosen (ties: the
-//                       lower index); their weights are the scores themselves, or the scores over their sum
-//   moe_combine_kernel  x <- x + sum of a token's `top` expert rows with their weights, in slot order
-//   moe_sort_kernel     the step's (token, slot) pairs ordered by expert, cut into row tiles of one expert each
+//                       lower index); their weights are the scores themselves, or the scores over their sum.  An optional correction per
+//                       expert is added to the score for the choice alone
+//   moe_combine_kernel  x <- x + sum of a token's `top` expert rows with their weights, in slot order (identity experts contribute the mixture's
+//                       input row), optionally with a shared expert's row, a second sublayer's row and a scale per column
+//   moe_sort_kernel     the step's (token, slot) pairs ordered by expert, cut into row tiles of one expert each; the pairs of experts without
+//                       matrices (identity experts, numbered behind the others) come last and get no tile
 //   moe_gemm_kernel     out[pair] = A[row of pair] . W_expert(pair)^T in IEEE fp32 for every tile, with the row products' fused epilogues
 //                       (gated activation on interleaved gate | up columns, plain store)
 //
@@ -35,6 +38,7 @@ struct MoeRouteArgs {
 	int group_kind;  // MOE_GROUP_TOP2_SUM (0) or MOE_GROUP_MAX: what a group scores
 	int renormalise; // 1: the chosen weights are divided by (their sum + renorm_eps)
 	float renorm_eps;
+	const float* correction; // (E) added to the scores where they are compared, not where they become weights; NULL: none.  Without groups
 };
 enum { MOE_SCORE_SIGMOID = 0, MOE_SCORE_SOFTMAX = 1 };
 enum { MOE_GROUP_TOP2_SUM = 0, MOE_GROUP_MAX = 1 };
@@ -119,11 +123,14 @@ __global__ void __launch_bounds__(256) moe_router_kernel(MoeRouteArgs a) {
 		float bv = -INFINITY;
 		int bi = -1;
 		for (int e = lane; e < a.E; e += 32)
-			if (flag[e] && (bi < 0 || sc[e] > bv)) { bv = sc[e]; bi = e; }
+			if (flag[e]) {
+				const float v = a.correction ? sc[e] + a.correction[e] : sc[e];
+				if (bi < 0 || v > bv) { bv = v; bi = e; }
+			}
 		warp_argmax(bv, bi);
 		if (lane == 0) {
 			a.idx[(size_t) t * a.top + r] = bi < 0 ? 0 : bi;
-			a.wgt[(size_t) t * a.top + r] = bi < 0 ? 0.f : bv;
+			a.wgt[(size_t) t * a.top + r] = bi < 0 ? 0.f : sc[bi];
 			if (bi >= 0) flag[bi] = 0;
 		}
 		__syncwarp();
@@ -145,18 +152,30 @@ struct MoeCombineArgs {
 	const float* x_in;   // (rows, width) or NULL
 	float* x_out;        // (rows, width); may be x_in
 	const SeqStep* step;
+	// identity experts: a pair whose expert number idx[pair] is n_experts or more contributes row ident[t] (the mixture's input)
+	const int* idx;      // (rows, top) or NULL: none
+	int n_experts;
+	const float* ident;  // (rows, width)
+	const float* base;   // (rows, width) added to the weighted sum (a shared expert's output), or NULL
+	const float* scale;  // (width) multiplies the sum, or NULL
+	const float* other;  // (rows, width) a sublayer beside the mixture: other_scale[c] * other[t][c] is added as well, or NULL
+	const float* other_scale;
 };
 // grid (tokens, column parts): a one-token step spreads its row over several CTAs
 static __global__ void moe_combine_kernel(MoeCombineArgs a) {
 	const int t = blockIdx.x;
 	if (t >= a.step->n) return;
 	for (int c = blockIdx.y * blockDim.x + threadIdx.x; c < a.width; c += gridDim.y * blockDim.x) {
+		const size_t at = (size_t) t * a.width + c;
 		float v = 0.f;
 		for (int p = 0; p < a.top; p++) {
 			const size_t pk = (size_t) t * a.top + p;
-			v = fmaf(a.wgt[pk], a.y[(a.part_row ? (size_t) a.part_row[pk] : pk) * a.ldy + c], v);
+			const float y = a.idx && a.idx[pk] >= a.n_experts ? a.ident[at] : a.y[(a.part_row ? (size_t) a.part_row[pk] : pk) * a.ldy + c];
+			v = fmaf(a.wgt[pk], y, v);
 		}
-		const size_t at = (size_t) t * a.width + c;
+		if (a.base) v += a.base[at];
+		if (a.scale) v *= a.scale[c];
+		if (a.other) v = fmaf(a.other_scale ? a.other_scale[c] : 1.f, a.other[at], v);
 		a.x_out[at] = a.x_in ? a.x_in[at] + v : v;
 	}
 }
@@ -177,6 +196,7 @@ struct MoeSortArgs {
 	int* n_tiles; // (1)
 	int* off;     // (E + 1) first place of every expert in `sorted`, or NULL
 	int* inv;     // (T * top) place of every pair in `sorted`, or NULL
+	int n_tiled;  // experts [n_tiled, E) get no tiles (they have no matrices); 0: every expert does
 };
 // one CTA; shared memory: 2 E + 1 ints
 static __global__ void moe_sort_kernel(MoeSortArgs a) {
@@ -192,7 +212,7 @@ static __global__ void moe_sort_kernel(MoeSortArgs a) {
 		int at = 0, nt = 0;
 		for (int e = 0; e < a.E; e++) {
 			off[e] = at;
-			for (int r = 0; r < cnt[e]; r += MOE_TM) {
+			for (int r = 0; r < cnt[e] && (a.n_tiled <= 0 || e < a.n_tiled); r += MOE_TM) {
 				a.tiles[3 * nt] = e;
 				a.tiles[3 * nt + 1] = at + r;
 				a.tiles[3 * nt + 2] = min(MOE_TM, cnt[e] - r);
@@ -238,6 +258,7 @@ struct MoeGemmArgs {
 	const int* idx; // (T, top) the pairs' experts
 	const SeqStep* step;
 	int top;
+	int n_experts;  // matvecs: pairs of experts from this number on have no matrix and are skipped; 0: none
 };
 
 // 64 x 64 x 16 tiles, 4 x 4 per thread, as rows_gemm_kernel; blockIdx.y walks the tile list
@@ -301,7 +322,7 @@ template <typename WT, int KS>
 __global__ void __launch_bounds__(256) moe_matvec_kernel(MoeGemmArgs a) {
 	__shared__ float red[8][2];
 	const int p = blockIdx.y;
-	if (p >= a.step->n * a.top) return;
+	if (p >= a.step->n * a.top || (a.n_experts > 0 && a.idx[p] >= a.n_experts)) return;
 	const int N = a.N, K = a.K;
 	const WT* W = reinterpret_cast<const WT*>(a.W) + (size_t) a.idx[p] * N * K;
 	const float* A = a.A + (size_t) (p / a.a_div) * a.lda;
@@ -366,6 +387,7 @@ static inline int launch_moe_router(const MoeRouteArgs& a, int rows, cudaStream_
 	if (a.E <= 0 || a.top <= 0 || a.top > a.E) return set_error(XALM_ERR_INVALID, "router: %d of %d experts", a.top, a.E);
 	if (a.n_groups > 1 && (a.E % a.n_groups || a.keep_groups <= 0 || a.keep_groups > a.n_groups || a.keep_groups * (a.E / a.n_groups) < a.top))
 		return set_error(XALM_ERR_INVALID, "router: %d groups, %d kept, cannot hold %d of %d experts", a.n_groups, a.keep_groups, a.top, a.E);
+	if (a.correction && a.n_groups > 1) return set_error(XALM_ERR_UNSUPPORTED, "router: a choice correction together with expert groups");
 	const size_t smem = moe_router_smem(a.K, a.E, a.n_groups);
 	if (a.w_bf16) moe_router_kernel<__nv_bfloat16><<<rows, 256, smem, s>>>(a);
 	else moe_router_kernel<float><<<rows, 256, smem, s>>>(a);
