@@ -283,29 +283,6 @@ RowsEpi residual_epi(Kb* m) { // x <- x + product
 	return e;
 }
 
-// What of a layer does not depend on the rest runs on the side stream (a branch of the one-token graph): the recurrences, which keep few SMs
-// busy for long, beside the attention and the feed-forward's products.  The side stream never runs a matrix product: the tensor-core path's
-// operand planes belong to the main stream.
-struct Fork {
-	Kb* m;
-	bool on;
-	cudaStream_t side() const { return on ? m->side : m->stream; }
-	int open() const {
-		if (!on) return XALM_OK;
-		XALM_CUDA_CHECK(cudaEventRecord(m->ev_fork, m->stream));
-		XALM_CUDA_CHECK(cudaStreamWaitEvent(m->side, m->ev_fork, 0));
-		return XALM_OK;
-	}
-	int mark() const { // the side branch ends here
-		if (on) XALM_CUDA_CHECK(cudaEventRecord(m->ev_join, m->side));
-		return XALM_OK;
-	}
-	int join() const {
-		if (on) XALM_CUDA_CHECK(cudaStreamWaitEvent(m->stream, m->ev_join, 0));
-		return XALM_OK;
-	}
-};
-
 // input projections on the main stream, then the recurrence on the fork's side
 int enqueue_gla(Kb* m, const Layer& L, const Run& R, int n, const Fork& fk, int* nl) {
 	const int H = L.H, d = L.d, dv = L.dv;

@@ -1,5 +1,5 @@
-// seq_family.cuh — the sequence engine shared by the model families that a config.json describes (Nabalix, Bolovik, Duletar, Kubolorn): what a
-// family does NOT write itself.
+// seq_family.cuh — the sequence engine shared by the model families that a config.json describes (Nabalix, Bolovik, Duletar, Kubolorn,
+// Mizerax): what a family does NOT write itself.
 //
 //   * tensors by name: the family lists what it reads (expect), the loader uploads them (any order, fp32 / fp16 / bf16), finalize
 //     turns them into device layouts (upload_rows: several matrices stacked or interleaved into one; upload_vec);
@@ -221,7 +221,7 @@ int tc_register(SeqModel* m, const WMat& wm, TcWeight* t) {
 // plane, or hi + lo with "seq_tc" = 2), fp32 accumulation, then the same epilogue as an elementwise kernel.
 int rows_product(SeqModel* m, const float* A, int lda, const void* W, const TcWeight* tw, int T, int N, int K, const RowsEpi& e, int* nl) {
 	if (m->use_tc && tw && tw->hi && T >= m->tc_min_rows && lda == K) {
-		if (e.kind == EPI_STORE && e.ldo % 4 == 0 && e.cap == 0.f && !e.mul) { // nothing to do to the product: the GEMM stores it itself
+		if (e.kind == EPI_STORE && e.ldo % 4 == 0 && e.cap == 0.f && !e.mul && !e.add) { // nothing to do to the product: the GEMM stores it itself
 			*nl += 2;
 			return tc_gemm(*tw, A, T, e.out, e.ldo, m->a_hi, m->a_lo, m->stream);
 		}
@@ -239,6 +239,30 @@ int rows_product(SeqModel* m, const float* A, int lda, const void* W, const TcWe
 		cudaError_t e_ = cudaGetLastError();                                                                        \
 		if (e_ != cudaSuccess) return set_error(XALM_ERR_CUDA, what " launch failed: %s", cudaGetErrorString(e_));   \
 	} while (0)
+
+// ---- side branch ----------------------------------------------------------------------------------------------------------------
+// What of a layer does not depend on the rest runs on the side stream (a branch of the one-token graph): a recurrence, which keeps few SMs
+// busy for long, or an attention beside the feed-forward's products.  The side stream never runs a matrix product: the tensor-core path's
+// operand planes belong to the main stream.
+struct Fork {
+	SeqModel* m;
+	bool on;
+	cudaStream_t side() const { return on ? m->side : m->stream; }
+	int open() const {
+		if (!on) return XALM_OK;
+		XALM_CUDA_CHECK(cudaEventRecord(m->ev_fork, m->stream));
+		XALM_CUDA_CHECK(cudaStreamWaitEvent(m->side, m->ev_fork, 0));
+		return XALM_OK;
+	}
+	int mark() const { // the side branch ends here
+		if (on) XALM_CUDA_CHECK(cudaEventRecord(m->ev_join, m->side));
+		return XALM_OK;
+	}
+	int join() const {
+		if (on) XALM_CUDA_CHECK(cudaStreamWaitEvent(m->stream, m->ev_join, 0));
+		return XALM_OK;
+	}
+};
 
 // ---- the step function ----------------------------------------------------------------------------------------------------------
 int check_ready(SeqModel* m) {

@@ -1,0 +1,166 @@
+// seq_moe.cuh — a mixture of experts as a sublayer of the config.json families: the expert matrices in the engine's layouts, the pass buffers,
+// and the kernels of moe_ops.cuh in order.
+//
+//   router -> [steps of a few tokens: one matvec per (token, slot) pair] or [sort by expert -> tiled fp32 products] or, for long passes of the
+//   16-bit mode, [sort -> gather -> every expert's rows through the tcgen05 GEMM on that expert's resident fp16 tiles]; the caller then joins
+//   each token's expert rows (moe_combine, with whatever else its layer adds there).
+//
+// A family says what differs between designs: how scores become choices and weights (MoeRouteArgs), the activation between an expert's two
+// products (RowsEpi), how many of the router's outputs are identity experts.
+#pragma once
+#include "moe_ops.cuh"
+#include "seq_family.cuh"
+
+namespace xalm {
+namespace seq {
+namespace {
+
+struct MoeWeights {
+	int E = 0, identity = 0; // experts with matrices; router outputs behind them that pass the input through
+	int top = 0, ff = 0;
+	int up_rows = 0;         // rows of an expert's first matrix: ff, or 2 ff when gate and up rows alternate
+	void *w_up = nullptr, *w_down = nullptr, *w_router = nullptr;
+	float* correction = nullptr; // (E + identity) or NULL
+	WMat m_up, m_down;
+	std::vector<TcWeight> t_up, t_down; // per expert, when long passes run on the tensor cores
+	bool on_tc(const SeqModel* m, int n) const { return m->use_tc && !t_up.empty() && n > 1 && n >= m->tc_min_rows; }
+};
+
+struct MoeBuffers { // of one pass, sized for the largest mixture of the model
+	size_t max_pairs = 0, max_hid = 0;
+	int max_tiles = 1, max_outputs = 1;
+	bool tc = false;
+	int *idx = nullptr, *sorted = nullptr, *tiles = nullptr, *ntiles = nullptr, *off = nullptr, *inv = nullptr, *h_off = nullptr;
+	float *wgt = nullptr, *hid = nullptr, *out = nullptr, *x = nullptr;
+};
+
+// tensors of `E` experts under prefix p ("<p>e0." ...): gate (when gated), up, down
+void moe_expect(SeqModel* m, const std::string& p, int E, int ff, bool gated) {
+	for (int e = 0; e < E; e++) {
+		const std::string pe = p + "e" + std::to_string(e) + ".";
+		if (gated) expect(m, pe + "gate", {ff, m->width}, true);
+		expect(m, pe + "up", {ff, m->width}, true);
+		expect(m, pe + "down", {m->width, ff}, true);
+	}
+}
+
+// device layouts of the experts (one after the other, gate / up rows alternating) and the router; grows what the buffers must hold
+int moe_upload(SeqModel* m, const std::string& p, bool gated, MoeWeights* L, MoeBuffers* b) {
+	std::vector<const HostTensor*> up, dn;
+	for (int e = 0; e < L->E; e++) {
+		const std::string pe = p + "e" + std::to_string(e) + ".";
+		if (gated) up.push_back(tensor_or_null(m, pe + "gate"));
+		up.push_back(tensor_or_null(m, pe + "up"));
+		dn.push_back(tensor_or_null(m, pe + "down"));
+	}
+	L->up_rows = gated ? 2 * L->ff : L->ff;
+	XALM_TRY(upload_rows(m, up, m->width, gated, &L->w_up, &L->m_up));
+	XALM_TRY(upload_rows(m, dn, L->ff, false, &L->w_down, &L->m_down));
+	XALM_TRY(upload_rows(m, {tensor_or_null(m, p + "router")}, m->width, false, &L->w_router, nullptr));
+	XALM_TRY(moe_prepare(m->width, L->E + L->identity, 0));
+	const size_t pairs = (size_t) m->chunk * L->top;
+	b->max_pairs = std::max(b->max_pairs, pairs);
+	b->max_hid = std::max(b->max_hid, pairs * L->ff);
+	b->max_tiles = std::max(b->max_tiles, moe_max_tiles((int) pairs, L->E));
+	b->max_outputs = std::max(b->max_outputs, L->E + L->identity);
+	return XALM_OK;
+}
+
+// a mixture whose expert shapes the GEMM takes keeps fp16 tiles per expert for its long passes
+int moe_tc_register(SeqModel* m, MoeWeights* L, MoeBuffers* b) {
+	const int W = m->width;
+	if (!m->use_tc || !tune("seq_moe_tc") || !tc_shape_ok(L->up_rows, W, L->up_rows) || !tc_shape_ok(W, L->ff, W)) return XALM_OK;
+	L->t_up.resize((size_t) L->E);
+	L->t_down.resize((size_t) L->E);
+	for (int e = 0; e < L->E; e++) {
+		WMat up = L->m_up, dn = L->m_down; // this expert's rows of the stacked matrices
+		up.rows = L->up_rows;
+		up.p0 = static_cast<const uint8_t*>(L->m_up.p0) + (size_t) e * L->up_rows * L->m_up.s0;
+		dn.rows = W;
+		dn.p0 = static_cast<const uint8_t*>(L->m_down.p0) + (size_t) e * W * L->m_down.s0;
+		XALM_TRY(tc_register(m, up, &L->t_up[(size_t) e]));
+		XALM_TRY(tc_register(m, dn, &L->t_down[(size_t) e]));
+	}
+	b->tc = true;
+	return XALM_OK;
+}
+
+int moe_alloc(SeqModel* m, MoeBuffers* b) {
+	if (!b->max_pairs) return XALM_OK;
+	const int W = m->width;
+	XALM_TRY(dev_alloc(m, &b->idx, b->max_pairs, true));
+	XALM_TRY(dev_alloc(m, &b->wgt, b->max_pairs, true));
+	XALM_TRY(dev_alloc(m, &b->sorted, b->max_pairs, true));
+	XALM_TRY(dev_alloc(m, &b->tiles, (size_t) 3 * b->max_tiles, true));
+	XALM_TRY(dev_alloc(m, &b->ntiles, 1, true));
+	XALM_TRY(dev_alloc(m, &b->hid, b->max_hid));
+	XALM_TRY(dev_alloc(m, &b->out, b->max_pairs * W));
+	if (b->tc) {
+		XALM_TRY(dev_alloc(m, &b->off, (size_t) b->max_outputs + 1, true));
+		XALM_TRY(dev_alloc(m, &b->inv, b->max_pairs, true));
+		XALM_TRY(dev_alloc(m, &b->x, b->max_pairs * W));
+		XALM_CUDA_CHECK(cudaMallocHost(&b->h_off, ((size_t) b->max_outputs + 1) * 4));
+	}
+	return XALM_OK;
+}
+
+void moe_free(MoeWeights* L) {
+	for (TcWeight& t : L->t_up) tc_weight_free(&t);
+	for (TcWeight& t : L->t_down) tc_weight_free(&t);
+}
+
+// Experts of n rows h (n, width) on the main stream.  `route` carries the scoring constants, `act` the epilogue of the first product (kind and
+// constants; out and ldo are set here).  Afterwards b.wgt and b.idx hold the choice and *ca names the expert rows for the caller's moe_combine.
+int moe_experts(SeqModel* m, const MoeWeights& L, const MoeBuffers& b, const float* h, int n, MoeRouteArgs route, RowsEpi act, MoeCombineArgs* ca, int* nl) {
+	cudaStream_t s = m->stream;
+	const int W = m->width, total = L.E + L.identity;
+	route.h = h; route.ldh = W; route.w = L.w_router; route.w_bf16 = m->w_bf16;
+	route.E = total; route.top = L.top; route.K = W; route.correction = L.correction;
+	route.idx = b.idx; route.wgt = b.wgt; route.step = m->d_step;
+	XALM_TRY(launch_moe_router(route, n, s));
+	(*nl)++;
+	const bool on_tc = L.on_tc(m, n);
+	if (on_tc || n * L.top > MOE_MATVEC_PAIRS) { // steps of a few tokens need no tile list
+		MoeSortArgs so = {b.idx, L.top, total, m->d_step, b.sorted, b.tiles, b.ntiles, b.off, b.inv, L.E};
+		XALM_TRY(launch_moe_sort(so, s));
+		(*nl)++;
+	}
+	act.ldo = L.ff;
+	if (on_tc) {
+		// Each expert's rows, gathered one after the other, go through the GEMM.  How many rows each expert got is read back first (one small copy
+		// and a wait per mixture layer and pass).
+		XALM_CUDA_CHECK(cudaMemcpyAsync(b.h_off, b.off, (size_t) (total + 1) * 4, cudaMemcpyDeviceToHost, s));
+		moe_gather_kernel<<<n * L.top, 256, 0, s>>>(h, W, L.top, b.sorted, m->d_step, L.top, W, b.x);
+		XALM_SEQ_LAUNCH_CHECK("moe_gather");
+		XALM_CUDA_CHECK(cudaStreamSynchronize(s));
+		for (int e = 0; e < L.E; e++) {
+			const int at = b.h_off[e], cnt = b.h_off[e + 1] - at;
+			if (cnt <= 0) continue;
+			XALM_TRY(tc_gemm(L.t_up[(size_t) e], b.x + (size_t) at * W, cnt, m->tc_out, L.up_rows, m->a_hi, m->a_lo, s));
+			act.out = b.hid + (size_t) at * L.ff;
+			XALM_TRY(launch_rows_epilogue(m->tc_out, L.up_rows, cnt, L.up_rows, act, s));
+			XALM_TRY(tc_gemm(L.t_down[(size_t) e], b.hid + (size_t) at * L.ff, cnt, b.out + (size_t) at * W, W, m->a_hi, m->a_lo, s));
+			*nl += 5;
+		}
+	} else {
+		MoeGemmArgs ga = {};
+		ga.A = h; ga.lda = W; ga.a_div = L.top; ga.W = L.w_up; ga.N = L.up_rows; ga.K = W;
+		ga.sorted = b.sorted; ga.tiles = b.tiles; ga.n_tiles = b.ntiles;
+		ga.idx = b.idx; ga.step = m->d_step; ga.top = L.top; ga.n_experts = L.E;
+		ga.e = act; ga.e.out = b.hid;
+		XALM_TRY(launch_moe_gemm(ga, m->w_bf16, n * L.top, L.E, s));
+		ga.A = b.hid; ga.lda = L.ff; ga.a_div = 1; ga.W = L.w_down; ga.N = W; ga.K = L.ff;
+		ga.e = RowsEpi();
+		ga.e.kind = EPI_STORE; ga.e.out = b.out; ga.e.ldo = W;
+		XALM_TRY(launch_moe_gemm(ga, m->w_bf16, n * L.top, L.E, s));
+		*nl += 2;
+	}
+	ca->y = b.out; ca->ldy = W; ca->top = L.top; ca->width = W; ca->wgt = b.wgt; ca->part_row = on_tc ? b.inv : nullptr;
+	ca->step = m->d_step;
+	if (L.identity) { ca->idx = b.idx; ca->n_experts = L.E; ca->ident = h; }
+	return XALM_OK;
+}
+
+} // namespace
+} // namespace seq
+} // namespace xalm
