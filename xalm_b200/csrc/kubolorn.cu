@@ -40,7 +40,7 @@
 #include "seq_family.cuh"
 
 #include "conv_ops.cuh"
-#include "moe_ops.cuh"
+#include "seq_moe.cuh"
 
 namespace xalm {
 namespace {
@@ -70,11 +70,11 @@ struct Layer { // weights and sizes; what a sequence holds lives in Run
 	float *conv_w = nullptr, *conv_b = nullptr, *dt_bias = nullptr, *A_log = nullptr, *D = nullptr, *s_norm = nullptr;
 	int n_in = 0, k_o = 0; // columns of the stacked input projection; rows the output projection reads
 	// feed-forward
-	int ff = 0, E = 0, top = 0;
-	void *w_in = nullptr, *w_o = nullptr, *w_up = nullptr, *w_down = nullptr, *w_router = nullptr;
+	int ff = 0; // dense
+	MoeWeights moe;
+	void *w_in = nullptr, *w_o = nullptr, *w_up = nullptr, *w_down = nullptr;
 	WMat m_in, m_o, m_up, m_down;
 	TcWeight t_in, t_o, t_up, t_down;
-	std::vector<TcWeight> t_eup, t_edown; // per expert, when the mixture's long passes run on the tensor cores
 	float *norm[2] = {nullptr, nullptr}, *canon[2] = {nullptr, nullptr};
 	long long bytes = 0, expert_bytes = 0; // what one run of the layer reads of its matrices; of that, one expert's share
 	int inner() const { return sH * sP; }
@@ -104,10 +104,7 @@ struct KubolornModel : SeqModel {
 	float *part_o = nullptr, *part_ml = nullptr;
 	unsigned* tickets = nullptr;
 	int part_cap = 0;
-	int *moe_idx = nullptr, *moe_sorted = nullptr, *moe_tiles = nullptr, *moe_ntiles = nullptr;
-	float *moe_wgt = nullptr, *moe_hid = nullptr, *moe_out = nullptr;
-	int *moe_off = nullptr, *moe_inv = nullptr, *h_off = nullptr;
-	float* moe_x = nullptr;
+	MoeBuffers moe;
 };
 typedef KubolornModel Kb;
 
@@ -235,17 +232,14 @@ int parse_config(SeqModel* sm, const char* json) {
 					expect(m, p + "mlp.down", {W, L.ff}, true);
 				} else if (kind == "moe") {
 					L.ff_kind = FF_MOE;
-					L.ff = geti(mlp->at("expert"), "ff");
+					L.moe.ff = geti(mlp->at("expert"), "ff");
 					const xjson::Value& r = mlp->at("router");
-					L.E = geti(r, "experts");
-					L.top = geti(r, "top");
-					if (L.ff <= 0 || L.E <= 0 || L.top <= 0 || L.top > L.E) return set_error(XALM_ERR_INVALID, "config: layer %zu: %d of %d experts of %d", li, L.top, L.E, L.ff);
-					for (int e = 0; e < L.E; e++) {
-						const std::string pe = p + "mlp.e" + std::to_string(e) + ".";
-						expect(m, pe + "up", {L.ff, W}, true);
-						expect(m, pe + "down", {W, L.ff}, true);
-					}
-					expect(m, p + "mlp.router", {L.E, W}, true);
+					L.moe.E = geti(r, "experts");
+					L.moe.top = geti(r, "top");
+					if (L.moe.ff <= 0 || L.moe.E <= 0 || L.moe.top <= 0 || L.moe.top > L.moe.E)
+						return set_error(XALM_ERR_INVALID, "config: layer %zu: %d of %d experts of %d", li, L.moe.top, L.moe.E, L.moe.ff);
+					moe_expect(m, p + "mlp.", L.moe.E, L.moe.ff, false);
+					expect(m, p + "mlp.router", {L.moe.E, W}, true);
 				} else return set_error(XALM_ERR_UNSUPPORTED, "config: layer %zu has feed-forward kind '%s'", li, kind.c_str());
 			}
 			expect(m, p + "canon1", {W, m->taps}, false);
@@ -367,58 +361,15 @@ int enqueue_parallel(Kb* m, const Layer& L, const Run& R, int n, const Fork& fk,
 }
 
 int enqueue_experts(Kb* m, const Layer& L, int n, int* nl) {
-	cudaStream_t s = m->stream;
-	const int W = m->width;
 	MoeRouteArgs ra = {};
-	ra.h = m->h2; ra.ldh = W; ra.w = L.w_router; ra.w_bf16 = m->w_bf16;
-	ra.E = L.E; ra.top = L.top; ra.K = W;
-	ra.idx = m->moe_idx; ra.wgt = m->moe_wgt; ra.step = m->d_step;
 	// the largest logits are the largest softmax scores; the chosen scores over their sum are the softmax over the chosen logits
 	ra.score_kind = MOE_SCORE_SOFTMAX; ra.group_kind = MOE_GROUP_MAX; ra.renormalise = 1; ra.renorm_eps = 0.f;
-	XALM_TRY(launch_moe_router(ra, n, s));
-	(*nl)++;
-	const bool on_tc = m->use_tc && !L.t_eup.empty() && n >= m->tc_min_rows;
-	const bool tiled = on_tc || n * L.top > MOE_MATVEC_PAIRS; // steps of a few tokens run one matvec per (token, slot) pair and need no tile list
-	if (tiled) {
-		MoeSortArgs so = {m->moe_idx, L.top, L.E, m->d_step, m->moe_sorted, m->moe_tiles, m->moe_ntiles, m->moe_off, m->moe_inv};
-		XALM_TRY(launch_moe_sort(so, s));
-		(*nl)++;
-	}
 	RowsEpi eu;
-	eu.kind = EPI_ACT; eu.act = ACT_RELU_SQUARED; eu.ldo = L.ff;
-	if (on_tc) {
-		// Long passes of the 16-bit mode: each expert's rows, gathered one after the other, go through the tcgen05 GEMM on that expert's
-		// resident fp16 tiles.  How many rows each expert got is read back first (one small copy and a wait per mixture layer and pass).
-		XALM_CUDA_CHECK(cudaMemcpyAsync(m->h_off, m->moe_off, (size_t) (L.E + 1) * 4, cudaMemcpyDeviceToHost, s));
-		moe_gather_kernel<<<n * L.top, 256, 0, s>>>(m->h2, W, L.top, m->moe_sorted, m->d_step, L.top, W, m->moe_x);
-		XALM_SEQ_LAUNCH_CHECK("moe_gather");
-		XALM_CUDA_CHECK(cudaStreamSynchronize(s));
-		for (int e = 0; e < L.E; e++) {
-			const int at = m->h_off[e], cnt = m->h_off[e + 1] - at;
-			if (cnt <= 0) continue;
-			XALM_TRY(tc_gemm(L.t_eup[(size_t) e], m->moe_x + (size_t) at * W, cnt, m->tc_out, L.ff, m->a_hi, m->a_lo, s));
-			eu.out = m->moe_hid + (size_t) at * L.ff;
-			XALM_TRY(launch_rows_epilogue(m->tc_out, L.ff, cnt, L.ff, eu, s));
-			XALM_TRY(tc_gemm(L.t_edown[(size_t) e], m->moe_hid + (size_t) at * L.ff, cnt, m->moe_out + (size_t) at * W, W, m->a_hi, m->a_lo, s));
-			*nl += 5;
-		}
-	} else {
-		MoeGemmArgs ga = {};
-		ga.A = m->h2; ga.lda = W; ga.a_div = L.top; ga.W = L.w_up; ga.N = L.ff; ga.K = W;
-		ga.sorted = m->moe_sorted; ga.tiles = m->moe_tiles; ga.n_tiles = m->moe_ntiles;
-		ga.idx = m->moe_idx; ga.step = m->d_step; ga.top = L.top;
-		ga.e = eu; ga.e.out = m->moe_hid;
-		XALM_TRY(launch_moe_gemm(ga, m->w_bf16, n * L.top, L.E, s));
-		ga.A = m->moe_hid; ga.lda = L.ff; ga.a_div = 1; ga.W = L.w_down; ga.N = W; ga.K = L.ff;
-		ga.e = RowsEpi();
-		ga.e.kind = EPI_STORE; ga.e.out = m->moe_out; ga.e.ldo = W;
-		XALM_TRY(launch_moe_gemm(ga, m->w_bf16, n * L.top, L.E, s));
-		*nl += 2;
-	}
+	eu.kind = EPI_ACT; eu.act = ACT_RELU_SQUARED;
 	MoeCombineArgs ca = {};
-	ca.y = m->moe_out; ca.ldy = W; ca.top = L.top; ca.width = W; ca.wgt = m->moe_wgt; ca.part_row = on_tc ? m->moe_inv : nullptr;
-	ca.x_in = m->x; ca.x_out = m->x; ca.step = m->d_step;
-	XALM_TRY(launch_moe_combine(ca, n, s));
+	ca.x_in = m->x; ca.x_out = m->x;
+	XALM_TRY(moe_experts(m, L.moe, m->moe, m->h2, n, ra, eu, &ca, nl));
+	XALM_TRY(launch_moe_combine(ca, n, m->stream));
 	(*nl)++;
 	return XALM_OK;
 }
@@ -483,9 +434,8 @@ int finalize(SeqModel* sm) {
 	const int W = m->width;
 	const size_t C = (size_t) m->chunk;
 	auto T = [&](const std::string& n) { return tensor_or_null(m, n); };
-	size_t max_proj = 4, max_att = 1, max_yssd = 1, max_ff = 1, max_hd = 1, max_h = 1, max_pairs = 0, max_moe_hid = 0, max_conv = 1;
-	int max_tiles = 1, max_norm_groups = m->groups, max_norm_width = W;
-	bool moe_tc = false;
+	size_t max_proj = 4, max_att = 1, max_yssd = 1, max_ff = 1, max_hd = 1, max_h = 1, max_conv = 1;
+	int max_norm_groups = m->groups, max_norm_width = W;
 	const size_t kelem = m->precision == XALM_PRECISION_F32 ? 4 : 2;
 	if (m->buckets) XALM_TRY(upload_rows(m, {T("bigram")}, W, false, &m->pair, nullptr));
 	XALM_TRY(upload_vec(m, "embed.norm", &m->embed_norm));
@@ -561,20 +511,8 @@ int finalize(SeqModel* sm) {
 			XALM_TRY(upload_rows(m, {T(p + "mlp.down")}, L.ff, false, &L.w_down, &L.m_down));
 			max_ff = std::max(max_ff, (size_t) L.ff);
 		} else if (L.ff_kind == FF_MOE) {
-			std::vector<const HostTensor*> up, dn;
-			for (int e = 0; e < L.E; e++) {
-				const std::string pe = p + "mlp.e" + std::to_string(e) + ".";
-				up.push_back(T(pe + "up"));
-				dn.push_back(T(pe + "down"));
-			}
-			XALM_TRY(upload_rows(m, up, W, false, &L.w_up, &L.m_up)); // all experts, one after the other
-			XALM_TRY(upload_rows(m, dn, L.ff, false, &L.w_down, &L.m_down));
-			XALM_TRY(upload_rows(m, {T(p + "mlp.router")}, W, false, &L.w_router, nullptr));
-			XALM_TRY(moe_prepare(W, L.E, 0));
-			L.expert_bytes = 2ll * L.ff * W * (m->w_bf16 ? 2 : 4);
-			max_pairs = std::max(max_pairs, C * L.top);
-			max_moe_hid = std::max(max_moe_hid, C * L.top * L.ff);
-			max_tiles = std::max(max_tiles, moe_max_tiles((int) C * L.top, L.E));
+			XALM_TRY(moe_upload(m, p + "mlp.", false, &L.moe, &m->moe));
+			L.expert_bytes = 2ll * L.moe.ff * W * (m->w_bf16 ? 2 : 4);
 		}
 		L.bytes = m->weight_bytes - bytes0;
 	}
@@ -586,21 +524,7 @@ int finalize(SeqModel* sm) {
 			XALM_TRY(tc_register(m, L.m_up, &L.t_up));
 			XALM_TRY(tc_register(m, L.m_down, &L.t_down));
 		}
-		// a mixture whose expert shapes the GEMM takes keeps fp16 tiles per expert for its long passes
-		if (L.ff_kind == FF_MOE && m->use_tc && tune("seq_moe_tc") && tc_shape_ok(L.ff, W, L.ff) && tc_shape_ok(W, L.ff, W)) {
-			L.t_eup.resize((size_t) L.E);
-			L.t_edown.resize((size_t) L.E);
-			for (int e = 0; e < L.E; e++) {
-				WMat up = L.m_up, dn = L.m_down; // this expert's rows of the stacked matrices
-				up.rows = L.ff;
-				up.p0 = static_cast<const uint8_t*>(L.m_up.p0) + (size_t) e * L.ff * L.m_up.s0;
-				dn.rows = W;
-				dn.p0 = static_cast<const uint8_t*>(L.m_down.p0) + (size_t) e * W * L.m_down.s0;
-				XALM_TRY(tc_register(m, up, &L.t_eup[(size_t) e]));
-				XALM_TRY(tc_register(m, dn, &L.t_edown[(size_t) e]));
-			}
-			moe_tc = true;
-		}
+		if (L.ff_kind == FF_MOE) XALM_TRY(moe_tc_register(m, &L.moe, &m->moe));
 	}
 	// what the sequence holds, per layer run
 	for (Run& R : m->runs) {
@@ -631,24 +555,7 @@ int finalize(SeqModel* sm) {
 	XALM_TRY(dev_alloc(m, &m->part_o, (size_t) m->part_cap * max_hd));
 	XALM_TRY(dev_alloc(m, &m->part_ml, (size_t) m->part_cap * 2 * max_h));
 	XALM_TRY(dev_alloc(m, &m->tickets, 8 * C, true));
-	if (max_pairs) {
-		XALM_TRY(dev_alloc(m, &m->moe_idx, max_pairs, true));
-		XALM_TRY(dev_alloc(m, &m->moe_wgt, max_pairs, true));
-		XALM_TRY(dev_alloc(m, &m->moe_sorted, max_pairs, true));
-		XALM_TRY(dev_alloc(m, &m->moe_tiles, (size_t) 3 * max_tiles, true));
-		XALM_TRY(dev_alloc(m, &m->moe_ntiles, 1, true));
-		XALM_TRY(dev_alloc(m, &m->moe_hid, max_moe_hid));
-		XALM_TRY(dev_alloc(m, &m->moe_out, max_pairs * W));
-		if (moe_tc) {
-			int max_e = 1;
-			for (const Layer& L : m->layers) max_e = std::max(max_e, L.E);
-			XALM_TRY(dev_alloc(m, &m->moe_off, (size_t) max_e + 1, true));
-			XALM_TRY(dev_alloc(m, &m->moe_inv, max_pairs, true));
-			XALM_TRY(dev_alloc(m, &m->moe_x, max_pairs * W));
-			XALM_CUDA_CHECK(cudaMallocHost(&m->h_off, ((size_t) max_e + 1) * 4));
-		}
-	}
-	return XALM_OK;
+	return moe_alloc(m, &m->moe);
 }
 
 int release(SeqModel* sm) {
@@ -675,7 +582,7 @@ long long active_bytes(SeqModel* sm, long long pos) {
 	std::vector<int> seen(m->layers.size(), 0);
 	for (const Run& R : m->runs) {
 		const Layer& L = m->layers[(size_t) R.layer];
-		const long long live = L.bytes - (L.ff_kind == FF_MOE ? (long long) (L.E - L.top) * L.expert_bytes : 0);
+		const long long live = L.bytes - (L.ff_kind == FF_MOE ? (long long) (L.moe.E - L.moe.top) * L.expert_bytes : 0);
 		b += seen[(size_t) R.layer]++ ? live : live - L.bytes;
 		if (L.mixer == MIX_GLA) b += 2ll * L.H * L.d * L.dv * 4;
 		else b += 2ll * L.sH * L.sN * L.sP * 4 + (pos + 1) * 2 * L.aG * L.ad * kelem;
@@ -696,10 +603,9 @@ void destroy(SeqModel* sm) {
 	Kb* m = static_cast<Kb*>(sm);
 	for (Layer& L : m->layers) {
 		for (TcWeight* t : {&L.t_in, &L.t_o, &L.t_up, &L.t_down}) tc_weight_free(t);
-		for (TcWeight& t : L.t_eup) tc_weight_free(&t);
-		for (TcWeight& t : L.t_edown) tc_weight_free(&t);
+		moe_free(&L.moe);
 	}
-	if (m->h_off) cudaFreeHost(m->h_off);
+	if (m->moe.h_off) cudaFreeHost(m->moe.h_off);
 	delete m;
 }
 

@@ -18,6 +18,7 @@ namespace {
 struct MoeWeights {
 	int E = 0, identity = 0; // experts with matrices; router outputs behind them that pass the input through
 	int top = 0, ff = 0;
+	int n_groups = 0, keep_groups = 0; // choice limited to the best expert groups (<= 1: not)
 	int up_rows = 0;         // rows of an expert's first matrix: ff, or 2 ff when gate and up rows alternate
 	void *w_up = nullptr, *w_down = nullptr, *w_router = nullptr;
 	float* correction = nullptr; // (E + identity) or NULL
@@ -57,7 +58,7 @@ int moe_upload(SeqModel* m, const std::string& p, bool gated, MoeWeights* L, Moe
 	XALM_TRY(upload_rows(m, up, m->width, gated, &L->w_up, &L->m_up));
 	XALM_TRY(upload_rows(m, dn, L->ff, false, &L->w_down, &L->m_down));
 	XALM_TRY(upload_rows(m, {tensor_or_null(m, p + "router")}, m->width, false, &L->w_router, nullptr));
-	XALM_TRY(moe_prepare(m->width, L->E + L->identity, 0));
+	XALM_TRY(moe_prepare(m->width, L->E + L->identity, L->n_groups));
 	const size_t pairs = (size_t) m->chunk * L->top;
 	b->max_pairs = std::max(b->max_pairs, pairs);
 	b->max_hid = std::max(b->max_hid, pairs * L->ff);
@@ -116,6 +117,7 @@ int moe_experts(SeqModel* m, const MoeWeights& L, const MoeBuffers& b, const flo
 	const int W = m->width, total = L.E + L.identity;
 	route.h = h; route.ldh = W; route.w = L.w_router; route.w_bf16 = m->w_bf16;
 	route.E = total; route.top = L.top; route.K = W; route.correction = L.correction;
+	route.n_groups = L.n_groups; route.keep_groups = L.keep_groups;
 	route.idx = b.idx; route.wgt = b.wgt; route.step = m->d_step;
 	XALM_TRY(launch_moe_router(route, n, s));
 	(*nl)++;
