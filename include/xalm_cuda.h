@@ -235,6 +235,28 @@ int xalm_cuda_qk_post(float* q_out, float* k_out, float* v_out, const float* pro
 int xalm_cuda_rows_act_bias(float* out, const float* x, const float* w, int T, int N, int K, int act, const float* bias, float act_pow, int w_bf16);
 int xalm_cuda_gated_group_norm(float* out, const float* y, const float* gate, const float* w, int T, int W, int groups, float eps, float out_scale, int ld_out);
 
+/* Mechanisms of unrotated attention and of mixtures with identity experts (fp32 host arrays in and out):
+ * layer_norm: (x - mean) / sqrt(mean squared deviation + eps) * w + b (b NULL: no bias), rows of W.
+ * embed_positions: out[t] = table[token_t] + positions[pos0 + t].
+ * head_norm_post: proj (T, H d + G d + G dv) = [q | k | v]; q and k heads over their root mean square times q_norm_w / k_norm_w (d); then q at
+ *   position p times 1 + temp_coef ln(floor((p + 1) / temp_every) + 1) (temp_every 0: as it is); k_out (ring, G d), v_out (ring, G dv) by row p % ring.
+ * biased_attention: causal softmax attention of scores scale q.k - slope[h] (i - j) (slope NULL: none), denominator + exp(sink[h]) (sink NULL:
+ *   none), times sigmoid(gate[t, h]) (T, H), NULL: no gate.  k (pos0 + T, G d), v (pos0 + T, G dv).
+ * moe_join: s = softmax(h w_router^T) over E experts and `identity` identity experts behind them; the `top` largest s + correction are chosen
+ *   (idx, wgt (T, top), wgt = s); out_pairs (T, top, K) the experts' outputs w_down (silu(w_gate h) . w_up h) (zero for identity experts);
+ *   x_io += scale . (sum wgt out + base) + other_scale . other, identity experts returning h.  base, scale, other, other_scale may be NULL.
+ * rows_add: out = x w^T + add. */
+int xalm_cuda_layer_norm(float* out, const float* x, const float* w, const float* b, int T, int W, float eps);
+int xalm_cuda_embed_positions(float* out, const int* tokens, int T, int pos0, const float* table, int vocab, const float* positions, int max_positions, int W);
+int xalm_cuda_head_norm_post(float* q_out, float* k_out, float* v_out, const float* proj, int T, int pos0, int H, int G, int d, int dv, const float* q_norm_w,
+                             const float* k_norm_w, float eps, int temp_every, float temp_coef, int ring);
+int xalm_cuda_biased_attention(float* out, const float* q, const float* gate, const float* k, const float* v, int T, int pos0, int H, int G, int d, int dv,
+                               float scale, const float* slope, const float* sink, int n_splits, int cache_bf16);
+int xalm_cuda_moe_join(float* x_io, float* out_pairs, int* idx, float* wgt, const float* h, const float* w_router, const float* correction, const float* w_gate,
+                       const float* w_up, const float* w_down, const float* base, const float* scale, const float* other, const float* other_scale, int T, int K,
+                       int E, int identity, int top, int ff, int w_bf16);
+int xalm_cuda_rows_add(float* out, const float* x, const float* w, const float* add, int T, int N, int K);
+
 /* Tensor parallel plumbing (no reference analogue; north star).  Rank 0 makes an id, the host side ships it to
  * the other ranks (torch.distributed / MPI / a file), every rank calls comm_init before finalize. */
 #define XALM_COMM_ID_BYTES 128

@@ -109,6 +109,12 @@ SYMBOLS = {
     "xalm_cuda_qk_post": (_i, [_vp] * 4 + [_i] * 5 + [_vp, _i, C.c_float, _i]),
     "xalm_cuda_rows_act_bias": (_i, [_vp] * 3 + [_i] * 4 + [_vp, C.c_float, _i]),
     "xalm_cuda_gated_group_norm": (_i, [_vp] * 4 + [_i] * 3 + [C.c_float, C.c_float, _i]),
+    "xalm_cuda_layer_norm": (_i, [_vp] * 4 + [_i, _i, C.c_float]),
+    "xalm_cuda_embed_positions": (_i, [_vp, _vp, _i, _i, _vp, _i, _vp, _i, _i]),
+    "xalm_cuda_head_norm_post": (_i, [_vp] * 4 + [_i] * 6 + [_vp, _vp, C.c_float, _i, C.c_float, _i]),
+    "xalm_cuda_biased_attention": (_i, [_vp] * 5 + [_i] * 6 + [C.c_float, _vp, _vp, _i, _i]),
+    "xalm_cuda_moe_join": (_i, [_vp] * 14 + [_i] * 7),
+    "xalm_cuda_rows_add": (_i, [_vp] * 4 + [_i] * 3),
 }
 PRECISION_BF16, PRECISION_F32 = 0, 1            # enum xalm_precision
 
@@ -510,4 +516,57 @@ def gated_group_norm(y, w, groups, gate=None, eps=1e-5, out_scale=0.0, ld_out=No
     ld_out = W if ld_out is None else ld_out
     out = np.zeros((T, ld_out), dtype=np.float32)
     check(lib().xalm_cuda_gated_group_norm(_p(out), _p(y), _pn(gate), _p(w), T, W, groups, eps, out_scale, ld_out))
+    return out
+
+
+def layer_norm(x, w, b=None, eps=1e-5):
+    x, w, b = _f(x), _f(w), _f(b)
+    out = np.empty_like(x)
+    check(lib().xalm_cuda_layer_norm(_p(out), _p(x), _p(w), _pn(b), x.shape[0], x.shape[1], eps))
+    return out
+
+
+def embed_positions(tokens, pos0, table, positions):
+    table, positions = _f(table), _f(positions)
+    tokens = np.ascontiguousarray(tokens, dtype=np.int32)
+    out = np.empty((len(tokens), table.shape[1]), dtype=np.float32)
+    check(lib().xalm_cuda_embed_positions(_p(out), _p(tokens), len(tokens), pos0, _p(table), table.shape[0], _p(positions), positions.shape[0], table.shape[1]))
+    return out
+
+
+def head_norm_post(proj, pos0, H, G, d, dv, q_norm_w, k_norm_w, eps=1e-5, temp_every=0, temp_coef=0.0, ring=None):
+    """Returns (q rows, K cache, V cache) with the caches row by row."""
+    proj, q_norm_w, k_norm_w = _f(proj), _f(q_norm_w), _f(k_norm_w)
+    T = proj.shape[0]
+    ring = pos0 + T if ring is None else ring
+    q, kc, vc = np.empty((T, H * d), dtype=np.float32), np.empty((ring, G * d), dtype=np.float32), np.empty((ring, G * dv), dtype=np.float32)
+    check(lib().xalm_cuda_head_norm_post(_p(q), _p(kc), _p(vc), _p(proj), T, pos0, H, G, d, dv, _p(q_norm_w), _p(k_norm_w), eps, temp_every, temp_coef, ring))
+    return q, kc, vc
+
+
+def biased_attention(q, k, v, pos0, H, G, d, dv, scale, slope=None, sink=None, gate=None, n_splits=1, cache_bf16=False):
+    q, k, v, slope, sink, gate = _f(q), _f(k), _f(v), _f(slope), _f(sink), _f(gate)
+    T = q.shape[0]
+    out = np.empty((T, H * dv), dtype=np.float32)
+    check(lib().xalm_cuda_biased_attention(_p(out), _p(q), _pn(gate), _p(k), _p(v), T, pos0, H, G, d, dv, scale, _pn(slope), _pn(sink), n_splits, int(cache_bf16)))
+    return out
+
+
+def moe_join(x, h, w_router, w_gate, w_up, w_down, top, correction=None, base=None, scale=None, other=None, other_scale=None, w_bf16=False):
+    """Returns (x after the join, idx (T, top), wgt (T, top)); router rows beyond the experts' number are identity experts."""
+    h, w_router, w_gate, w_up, w_down = _f(h), _f(w_router), _f(w_gate), _f(w_up), _f(w_down)
+    correction, base, scale, other, other_scale = (_f(a) for a in (correction, base, scale, other, other_scale))
+    T, K = h.shape
+    E, ff = w_gate.shape[0], w_gate.shape[1]
+    idx, wgt, pairs = np.empty((T, top), dtype=np.int32), np.empty((T, top), dtype=np.float32), np.empty((T, top, K), dtype=np.float32)
+    xo = np.array(x, dtype=np.float32, copy=True)
+    check(lib().xalm_cuda_moe_join(_p(xo), _p(pairs), _p(idx), _p(wgt), _p(h), _p(w_router), _pn(correction), _p(w_gate), _p(w_up), _p(w_down), _pn(base),
+                                   _pn(scale), _pn(other), _pn(other_scale), T, K, E, w_router.shape[0] - E, top, ff, int(w_bf16)))
+    return xo, idx, wgt
+
+
+def rows_add(x, w, add):
+    x, w, add = _f(x), _f(w), _f(add)
+    out = np.empty((x.shape[0], w.shape[0]), dtype=np.float32)
+    check(lib().xalm_cuda_rows_add(_p(out), _p(x), _p(w), _p(add), x.shape[0], w.shape[0], x.shape[1]))
     return out

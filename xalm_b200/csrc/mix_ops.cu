@@ -62,7 +62,7 @@ uint16_t bf16_bits(float f) {
 
 static int swa_attention_op(float* out, const float* q, const float* gate, const float* k, const float* v, int T, int pos0, int H, int G, int d, int dv,
                             int window, int keep_first, float scale, float softcap, const float* r1, const float* r2, const float* talk, int ring, int n_splits,
-                            int cache_bf16, const float* sink = nullptr, float out_scale = 0.f) {
+                            int cache_bf16, const float* sink = nullptr, float out_scale = 0.f, const float* slope = nullptr, bool gate_per_head = false) {
 	if (!out || !q || !k || !v || T <= 0 || pos0 < 0 || H <= 0 || G <= 0 || H % G || d <= 0 || dv <= 0 || window <= 0 || n_splits < 1 || keep_first < 0)
 		return set_error(XALM_ERR_INVALID, "swa_attention: bad argument");
 	const int n = pos0 + T;
@@ -92,9 +92,10 @@ static int swa_attention_op(float* out, const float* q, const float* gate, const
 	const SeqStep st = {pos0, T};
 	SwaArgs a = {};
 	a.q = pool.put(q, (size_t) T * H * d);
-	a.gate = pool.put(gate, (size_t) T * H * dv);
+	a.ldg = gate_per_head ? H : H * dv;
+	a.gate = pool.put(gate, (size_t) T * a.ldg); a.gate_per_head = gate_per_head;
 	a.ldq = H * d; a.q_off = 0; a.g_off = 0;
-	a.ldg = H * dv;
+	a.slope = pool.put(slope, (size_t) H);
 	a.kc = pool.put(kr.data(), kr.size());
 	a.vc = pool.put(vr.data(), vr.size());
 	a.ring = ring; a.keep_first = keep_first; a.H = H; a.G = G; a.d = d; a.dv = dv; a.window = window; a.scale = scale; a.softcap = softcap;
@@ -247,7 +248,7 @@ int xalm_cuda_group_norm_residual(float* x_out, float* avg_out, const float* y, 
 
 static int qkv_post_op(float* q_out, float* k_out, float* v_out, const float* proj, int T, int pos0, int H, int G, int d, int dv, const float* bq,
                        const float* bk, const float* bv, const float* freq, int rot_half, int norm_qk, int norm_v, float eps, int keep_first, int ring,
-                       float rot_mag, int v_from_k) {
+                       float rot_mag, int v_from_k, const float* q_norm_w = nullptr, const float* k_norm_w = nullptr, int temp_every = 0, float temp_coef = 0.f) {
 	if (!q_out || !k_out || !v_out || !proj || T <= 0 || pos0 < 0 || H <= 0 || G <= 0 || d <= 0 || dv <= 0 || 2 * rot_half > d || keep_first < 0 || ring < 1)
 		return set_error(XALM_ERR_INVALID, "qkv_post: bad argument");
 	Pool pool;
@@ -261,6 +262,7 @@ static int qkv_post_op(float* q_out, float* k_out, float* v_out, const float* pr
 	a.bq = pool.put(bq, (size_t) H * d); a.bk = pool.put(bk, (size_t) G * d); a.bv = pool.put(bv, (size_t) G * dv);
 	a.freq = rot_half ? pool.put(freq, (size_t) rot_half) : nullptr; a.rot_half = rot_half;
 	a.norm_qk = norm_qk; a.norm_v = norm_v; a.eps = eps;
+	a.q_norm_w = pool.put(q_norm_w, (size_t) d); a.k_norm_w = pool.put(k_norm_w, (size_t) d); a.temp_every = temp_every; a.temp_coef = temp_coef;
 	float* kc = pool.raw<float>((size_t) slots * G * d);
 	float* vc = pool.raw<float>((size_t) slots * G * dv);
 	a.kc = kc; a.vc = vc; a.cache_f32 = 1; a.keep_first = keep_first; a.ring = ring;
@@ -280,6 +282,12 @@ static int qkv_post_op(float* q_out, float* k_out, float* v_out, const float* pr
 int xalm_cuda_qkv_post(float* q_out, float* k_out, float* v_out, const float* proj, int T, int pos0, int H, int G, int d, int dv, const float* bq,
                        const float* bk, const float* bv, const float* freq, int rot_half, int norm_qk, int norm_v, float eps, int keep_first, int ring) {
 	return qkv_post_op(q_out, k_out, v_out, proj, T, pos0, H, G, d, dv, bq, bk, bv, freq, rot_half, norm_qk, norm_v, eps, keep_first, ring, 0.f, 0);
+}
+int xalm_cuda_head_norm_post(float* q_out, float* k_out, float* v_out, const float* proj, int T, int pos0, int H, int G, int d, int dv, const float* q_norm_w,
+                             const float* k_norm_w, float eps, int temp_every, float temp_coef, int ring) {
+	if (!q_norm_w || !k_norm_w || temp_every < 0) return set_error(XALM_ERR_INVALID, "head_norm_post: bad argument");
+	return qkv_post_op(q_out, k_out, v_out, proj, T, pos0, H, G, d, dv, nullptr, nullptr, nullptr, nullptr, 0, 1, 0, eps, 0, ring, 0.f, 0, q_norm_w, k_norm_w,
+	                   temp_every, temp_coef);
 }
 int xalm_cuda_qk_post(float* q_out, float* k_out, float* v_out, const float* proj, int T, int pos0, int H, int G, int d, const float* freq, int rot_half,
                       float rot_mag, int ring) {
@@ -332,9 +340,14 @@ int xalm_cuda_delta_rule(float* out, float* state, float* conv_state, const floa
 
 } // extern "C"
 
+// what a mixture may have beside its experts: router outputs that return the input, a correction of the choice, rows and scales of the join
+struct MoeExtras {
+	int identity = 0;
+	const float *correction = nullptr, *base = nullptr, *scale = nullptr, *other = nullptr, *other_scale = nullptr;
+};
 static int moe_ffn_op(float* out_pairs, int* idx, float* wgt, const float* h, const float* w_router, const float* w_gate, const float* w_up,
                       const float* w_down, int T, int K, int E, int top, int ff, int n_groups, int keep_groups, int act, int w_bf16, int score_kind,
-                      int group_kind, int renormalise, float limit, float* x_io) {
+                      int group_kind, int renormalise, float limit, float* x_io, const MoeExtras& ex = MoeExtras()) {
 	if (!out_pairs || !idx || !wgt || !h || !w_router || !w_gate || !w_up || !w_down || T <= 0 || K <= 0 || E <= 0 || top <= 0 || ff <= 0)
 		return set_error(XALM_ERR_INVALID, "moe_ffn: bad argument");
 	Pool pool;
@@ -353,24 +366,25 @@ static int moe_ffn_op(float* out_pairs, int* idx, float* wgt, const float* h, co
 	};
 	const SeqStep st = {0, T};
 	const SeqStep* d_st = pool.put(&st, 1);
-	const int P = T * top, max_tiles = moe_max_tiles(P, E);
+	const int P = T * top, total = E + ex.identity, max_tiles = moe_max_tiles(P, E);
 	MoeRouteArgs ra = {};
-	ra.h = pool.put(h, (size_t) T * K); ra.ldh = K; ra.w = put_w(w_router, (size_t) E * K); ra.w_bf16 = w_bf16;
-	ra.E = E; ra.top = top; ra.K = K; ra.n_groups = n_groups; ra.keep_groups = keep_groups;
+	ra.h = pool.put(h, (size_t) T * K); ra.ldh = K; ra.w = put_w(w_router, (size_t) total * K); ra.w_bf16 = w_bf16;
+	ra.correction = pool.put(ex.correction, (size_t) total);
+	ra.E = total; ra.top = top; ra.K = K; ra.n_groups = n_groups; ra.keep_groups = keep_groups;
 	ra.idx = pool.raw<int>((size_t) P); ra.wgt = pool.raw<float>((size_t) P); ra.step = d_st;
 	ra.score_kind = score_kind; ra.group_kind = group_kind; ra.renormalise = renormalise; ra.renorm_eps = 1e-20f;
-	MoeSortArgs so = {ra.idx, top, E, d_st, pool.raw<int>((size_t) P), pool.raw<int>((size_t) 3 * max_tiles), pool.raw<int>(1), nullptr, nullptr};
+	MoeSortArgs so = {ra.idx, top, total, d_st, pool.raw<int>((size_t) P), pool.raw<int>((size_t) 3 * max_tiles), pool.raw<int>(1), nullptr, nullptr, E};
 	MoeGemmArgs ga = {};
 	ga.A = ra.h; ga.lda = K; ga.a_div = top; ga.W = put_w(gu.data(), gu.size()); ga.N = 2 * ff; ga.K = K;
 	ga.sorted = so.sorted; ga.tiles = so.tiles; ga.n_tiles = so.n_tiles;
-	ga.idx = ra.idx; ga.step = d_st; ga.top = top;
+	ga.idx = ra.idx; ga.step = d_st; ga.top = top; ga.n_experts = E;
 	float* hid = pool.raw<float>((size_t) P * ff);
 	float* outp = pool.raw<float>((size_t) P * K);
 	ga.e.kind = EPI_GLU; ga.e.glu_act = act; ga.e.out = hid; ga.e.ldo = ff; ga.e.limit = limit;
 	void* d_down = put_w(w_down, (size_t) E * K * ff);
 	if (!d_st || !ra.h || !ra.w || !ra.idx || !ra.wgt || !so.sorted || !so.tiles || !so.n_tiles || !ga.W || !hid || !outp || !d_down)
 		return set_error(XALM_ERR_CUDA, "moe_ffn: device allocation failed");
-	XALM_TRY(moe_prepare(K, E, n_groups));
+	XALM_TRY(moe_prepare(K, total, n_groups));
 	XALM_TRY(launch_moe_router(ra, T, nullptr));
 	XALM_TRY(launch_moe_sort(so, nullptr));
 	XALM_TRY(launch_moe_gemm(ga, w_bf16 != 0, P, E, nullptr));
@@ -382,6 +396,11 @@ static int moe_ffn_op(float* out_pairs, int* idx, float* wgt, const float* h, co
 	if (x_io) { // the residual stream takes the weighted sum of each token's rows
 		if (!d_x) return set_error(XALM_ERR_CUDA, "moe_ffn: device allocation failed");
 		MoeCombineArgs ca = {outp, K, top, K, ra.wgt, nullptr, d_x, d_x, d_st};
+		if (ex.identity) { ca.idx = ra.idx; ca.n_experts = E; ca.ident = ra.h; }
+		ca.base = pool.put(ex.base, (size_t) T * K);
+		ca.scale = pool.put(ex.scale, (size_t) K);
+		ca.other = pool.put(ex.other, (size_t) T * K);
+		ca.other_scale = pool.put(ex.other_scale, (size_t) K);
 		XALM_TRY(launch_moe_combine(ca, T, nullptr));
 	}
 	XALM_TRY(finish("moe_ffn"));
@@ -404,6 +423,16 @@ int xalm_cuda_moe_ffn_routed(float* out_pairs, int* idx, float* wgt, float* x_io
                              int w_bf16, int score_kind, int group_kind, int renormalise, float limit) {
 	return moe_ffn_op(out_pairs, idx, wgt, h, w_router, w_gate, w_up, w_down, T, K, E, top, ff, n_groups, keep_groups, act, w_bf16, score_kind, group_kind,
 	                  renormalise, limit, x_io);
+}
+
+int xalm_cuda_moe_join(float* x_io, float* out_pairs, int* idx, float* wgt, const float* h, const float* w_router, const float* correction, const float* w_gate,
+                       const float* w_up, const float* w_down, const float* base, const float* scale, const float* other, const float* other_scale, int T, int K,
+                       int E, int identity, int top, int ff, int w_bf16) {
+	if (!x_io || identity < 0) return set_error(XALM_ERR_INVALID, "moe_join: bad argument");
+	MoeExtras ex;
+	ex.identity = identity; ex.correction = correction; ex.base = base; ex.scale = scale; ex.other = other; ex.other_scale = other_scale;
+	return moe_ffn_op(out_pairs, idx, wgt, h, w_router, w_gate, w_up, w_down, T, K, E, top, ff, 0, 0, GLU_SILU, w_bf16, MOE_SCORE_SOFTMAX, MOE_GROUP_MAX, 0,
+	                  INFINITY, x_io, ex);
 }
 
 int xalm_cuda_retention(float* out, float* state, const float* q, const float* k, const float* v, const float* gate, int T, int pos0, int H, int d, int dv,
@@ -574,6 +603,56 @@ int xalm_cuda_sink_attention(float* out, const float* q, const float* k, const f
                              const float* sink, float out_scale, int n_splits, int cache_bf16) {
 	return swa_attention_op(out, q, nullptr, k, v, T, pos0, H, G, d, dv, 0x7fffffff, 0, scale, 0.f, nullptr, nullptr, nullptr, pos0 + T, n_splits, cache_bf16, sink,
 	                        out_scale);
+}
+
+int xalm_cuda_biased_attention(float* out, const float* q, const float* gate, const float* k, const float* v, int T, int pos0, int H, int G, int d, int dv,
+                               float scale, const float* slope, const float* sink, int n_splits, int cache_bf16) {
+	return swa_attention_op(out, q, gate, k, v, T, pos0, H, G, d, dv, 0x7fffffff, 0, scale, 0.f, nullptr, nullptr, nullptr, pos0 + T, n_splits, cache_bf16, sink, 0.f,
+	                        slope, true);
+}
+
+int xalm_cuda_layer_norm(float* out, const float* x, const float* w, const float* b, int T, int W, float eps) {
+	if (!out || !x || !w || T <= 0 || W <= 0) return set_error(XALM_ERR_INVALID, "layer_norm: bad argument");
+	Pool pool;
+	const float *d_x = pool.put(x, (size_t) T * W), *d_w = pool.put(w, (size_t) W), *d_b = pool.put(b, (size_t) W);
+	float* d_out = pool.raw<float>((size_t) T * W);
+	if (!d_x || !d_w || !d_out || (b && !d_b)) return set_error(XALM_ERR_CUDA, "layer_norm: device allocation failed");
+	XALM_TRY(layer_norm_prepare(W));
+	XALM_TRY(launch_layer_norm(d_x, W, d_w, d_b, eps, W, d_out, T, nullptr));
+	XALM_TRY(finish("layer_norm"));
+	XALM_CUDA_CHECK(cudaMemcpy(out, d_out, (size_t) T * W * 4, cudaMemcpyDeviceToHost));
+	return XALM_OK;
+}
+
+int xalm_cuda_embed_positions(float* out, const int* tokens, int T, int pos0, const float* table, int vocab, const float* positions, int max_positions, int W) {
+	if (!out || !tokens || !table || !positions || T <= 0 || vocab <= 0 || W <= 0 || pos0 < 0 || pos0 + T > max_positions)
+		return set_error(XALM_ERR_INVALID, "embed_positions: bad argument");
+	for (int t = 0; t < T; t++)
+		if (tokens[t] < 0 || tokens[t] >= vocab) return set_error(XALM_ERR_INVALID, "embed_positions: token %d out of range", tokens[t]);
+	Pool pool;
+	const SeqStep st = {pos0, T, -1};
+	const float *d_table = pool.put(table, (size_t) vocab * W), *d_pos = pool.put(positions, (size_t) max_positions * W);
+	const int* d_tok = pool.put(tokens, (size_t) T);
+	const SeqStep* d_st = pool.put(&st, 1);
+	float* d_out = pool.raw<float>((size_t) T * W);
+	if (!d_table || !d_pos || !d_tok || !d_st || !d_out) return set_error(XALM_ERR_CUDA, "embed_positions: device allocation failed");
+	embed_streams_kernel<float><<<T, norm_threads(W)>>>(d_table, d_tok, W, 1, (size_t) T * W, d_out, 1.f, d_pos, d_st);
+	XALM_TRY(finish("embed_positions"));
+	XALM_CUDA_CHECK(cudaMemcpy(out, d_out, (size_t) T * W * 4, cudaMemcpyDeviceToHost));
+	return XALM_OK;
+}
+
+int xalm_cuda_rows_add(float* out, const float* x, const float* w, const float* add, int T, int N, int K) {
+	if (!out || !x || !w || !add || T <= 0 || N <= 0 || K <= 0) return set_error(XALM_ERR_INVALID, "rows_add: bad argument");
+	Pool pool;
+	const float *d_x = pool.put(x, (size_t) T * K), *d_w = pool.put(w, (size_t) N * K), *d_add = pool.put(add, (size_t) T * N);
+	RowsEpi e;
+	e.kind = EPI_STORE; e.out = pool.raw<float>((size_t) T * N); e.ldo = N; e.add = d_add; e.lda = N;
+	if (!d_x || !d_w || !d_add || !e.out) return set_error(XALM_ERR_CUDA, "rows_add: device allocation failed");
+	XALM_TRY(launch_rows(d_x, K, d_w, false, T, N, K, e, nullptr));
+	XALM_TRY(finish("rows_add"));
+	XALM_CUDA_CHECK(cudaMemcpy(out, e.out, (size_t) T * N * 4, cudaMemcpyDeviceToHost));
+	return XALM_OK;
 }
 
 int xalm_cuda_norm_conv(float* out, float* hist, const float* x, int T, int W, int groups, int taps, int readers, const float* w, const float* cw, float eps) {
