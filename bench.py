@@ -582,6 +582,47 @@ def build_kubolorn(z: dict, seed: int, max_tokens: int, stream):
     return m
 
 
+def mizerax_config(z: dict) -> dict:
+    """Every layer: attention (no window, distance bias, head norms, query temperature, head gates) beside a mixture of 16 gated experts of ff / 4
+    of which 4 are chosen, 2 identity experts and a shared expert of ff / 4.  The second half of the layers is one pass over a loop, so that
+    as many layers run as in the other families' models of the size and all read weights of their own."""
+    att = {"heads": z["heads"], "kv_heads": z["kv_heads"], "dim": z["head_dim"], "vdim": z["head_dim"], "scale": z["head_dim"] ** -0.5,
+           "q_temp": {"coef": 0.2, "every": 1024}}
+    moe = {"kind": "moe", "expert": {"ff": z["ff"] // 4}, "router": {"experts": 16, "top": 4, "identity": 2}, "shared": {"ff": z["ff"] // 4}}
+    return {"architecture": "Mizerax", "vocab": z["vocab"], "width": z["width"], "max_positions": 4096, "norm": {"eps": 1e-6}, "residual_mult": 0.5,
+            "layers": [{"type": "attention", "mixer": att, "mlp": moe}] * z["layers"],
+            "loop": {"start": z["layers"] // 2, "stop": z["layers"], "times": 1}}
+
+
+def build_mizerax(z: dict, seed: int, max_tokens: int, stream):
+    """Random bf16 weights, uploaded tensor by tensor as the backend names them."""
+    import ctypes as C
+    import json
+    from xalm_b200 import capi, safetensors_io as ST, types as T
+    from xalm_b200.model import Model
+    m = Model._from_json_text(json.dumps(mizerax_config(z)), {})
+    L = capi.lib()
+    h = C.c_void_p()
+    capi.check(L.xalm_cuda_create_json(m.config["json"].encode(), 0, max_tokens, capi.PRECISION_BF16, C.byref(h)))
+    m._h = h
+    capi.check(L.xalm_cuda_set_stream(h, C.c_void_p(stream)))
+    rng = np.random.default_rng(seed)
+    for name, shape in m.expected_tensors().items():
+        leaf = name.split(".")[-1]
+        if name in ("embed", "pos"):
+            a = rng.standard_normal(shape, dtype=np.float32) * np.float32(1.0 if name == "embed" else 0.3)
+        elif len(shape) == 2:
+            a = rng.standard_normal(shape, dtype=np.float32) * np.float32((2.0 if leaf == "router" else 1.0) / np.sqrt(shape[1]))
+        elif leaf in ("b", "correction"):
+            a = (0.1 if leaf == "b" else 0.02) * rng.standard_normal(shape, dtype=np.float32)
+        else:
+            a = 1.0 + 0.1 * rng.standard_normal(shape, dtype=np.float32)
+        m.upload(name, T.BF16, shape, ST.f32_to_bf16_bits(a).view(np.uint8).reshape(-1))
+    capi.check(L.xalm_cuda_finalize(h))
+    m.config["vocab_size"] = z["vocab"]
+    return m
+
+
 def run_family_workload(args, fams=("nabalix", "llama")):
     """Prefill and one-token-step throughput of config.json families beside one another and beside the Llama family at equal layer sizes
     (bf16 weights, random), device-timed with CUDA events on the launching stream.  One JSON line; `value` is the first family's decode rate
@@ -606,7 +647,8 @@ def run_family_workload(args, fams=("nabalix", "llama")):
             for fam in fams:
                 if fam != "llama":
                     capi.tune("seq_chunk", args.seq_chunk)  # positions per pass of a prompt (the Llama arm takes the prompt in one pass)
-                    m = {"nabalix": build_nabalix, "bolovik": build_bolovik, "duletar": build_duletar, "kubolorn": build_kubolorn}[fam](z, args.seed, ctx, stream.cuda_stream)
+                    m = {"nabalix": build_nabalix, "bolovik": build_bolovik, "duletar": build_duletar, "kubolorn": build_kubolorn,
+                         "mizerax": build_mizerax}[fam](z, args.seed, ctx, stream.cuda_stream)
                 else:
                     m, _ = build_model_streaming(llama_full, llama_cfg, T.BF16, args.seed, False, stream=stream.cuda_stream)
                     capi.tune("prefill_split", 1)        # plain fp16 operands, the counterpart of the one-plane path
@@ -667,14 +709,15 @@ def main():
     ap.add_argument("--past-window", action="store_true",
                     help="also time steps at positions >= ctx: the KV ring is full (kv_len = ctx), 2 attention sinks active (infer.cpp:608-613)")
     ap.add_argument("--no-prefill", action="store_true", help="skip the perplexity-mode summary appended to the decode line at N=1")
-    ap.add_argument("--workload", default="decode", choices=["decode", "perplexity", "families", "bolovik", "duletar", "kubolorn"],
+    ap.add_argument("--workload", default="decode", choices=["decode", "perplexity", "families", "bolovik", "duletar", "kubolorn", "mizerax"],
                     help="decode = BASELINE config[1] (the headline metric); perplexity = config[2]: batched prefill of a 4k-token input; "
                          "families = prefill and one-token-step throughput of the Nabalix family beside the Llama family at equal layer sizes; "
                          "bolovik = the same for the Bolovik family beside the Nabalix and Llama families; "
                          "duletar = the same for the Duletar family beside the Bolovik family; "
-                         "kubolorn = the same for the Kubolorn family beside the Bolovik family")
-    ap.add_argument("--arms", default="", help="bolovik / duletar / kubolorn workloads: which families run, the first one is the headline "
-                                               "(default bolovik,nabalix,llama / duletar,bolovik / kubolorn,bolovik)")
+                         "kubolorn = the same for the Kubolorn family beside the Bolovik family; "
+                         "mizerax = the same for the Mizerax family beside the Bolovik and Kubolorn families")
+    ap.add_argument("--arms", default="", help="bolovik / duletar / kubolorn / mizerax workloads: which families run, the first one is the headline "
+                                               "(default bolovik,nabalix,llama / duletar,bolovik / kubolorn,bolovik / mizerax,bolovik,kubolorn)")
     ap.add_argument("--seq-chunk", type=int, default=1024, help="families workload: positions per pass of a Nabalix prompt")
     ap.add_argument("--sizes", default="w1024,w2048,w4096", help="families workload: which of " + ",".join(FAMILY_SIZES))
     ap.add_argument("--tokens", type=int, default=4096, help="perplexity workload: tokens per step")
@@ -685,9 +728,10 @@ def main():
     if args.workload == "perplexity":
         run_perplexity_workload(args)
         return
-    if args.workload in ("families", "bolovik", "duletar", "kubolorn"):
+    if args.workload in ("families", "bolovik", "duletar", "kubolorn", "mizerax"):
         if not args.arms:
-            args.arms = {"duletar": "duletar,bolovik", "kubolorn": "kubolorn,bolovik"}.get(args.workload, "bolovik,nabalix,llama")
+            args.arms = {"duletar": "duletar,bolovik", "kubolorn": "kubolorn,bolovik",
+                         "mizerax": "mizerax,bolovik,kubolorn"}.get(args.workload, "bolovik,nabalix,llama")
         if args.steps == 256:
             args.steps = 64
         if args.tokens == 4096:

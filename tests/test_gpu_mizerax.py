@@ -322,6 +322,34 @@ def test_tensor_core_passes_match_the_fp32_kernels():
     rows_within(outputs[1], outputs[0], BF16_TOL)
 
 
+@pytest.mark.parametrize("E,top,identity,ff", [(2, 2, 1, 192), (7, 3, 0, 64), (40, 8, 4, 64), (1, 1, 3, 320)])
+def test_experts_of_long_passes_share_one_grouped_product(E, top, identity, ff):
+    """Few experts with several row tiles each (the last one partly filled), many experts with a handful of rows, matrices of more than one
+    column tile, passes in which most pairs are identity experts: against the oracle, and the two-plane operands against the fp32 tiles."""
+    cfg = O.make_config(vocab=50, width=128, max_positions=512, mult=0.5, layers=[A(2, 1, 16, 16, 0.25, None, mlp=M(ff, E, top, identity=identity))])
+    W = O.random_weights(cfg, seed=E)
+    if E == 1:
+        W["l0.mlp.correction"] = np.array([0.0, 0.6, 0.0, 0.0])
+    tokens = np.random.default_rng(E).integers(0, 50, 410).tolist()
+    logits = O.forward(cfg, W, tokens, {})
+    out = {}
+    for tc, moe_tc in ((1, 1), (2, 1), (2, 0)):
+        capi.tune("seq_tc", tc)
+        capi.tune("seq_moe_tc", moe_tc)
+        try:
+            m = on_gpu(cfg, W, capi.PRECISION_BF16, chunk=512, max_tokens=512)
+        finally:
+            capi.tune("seq_tc", 1)
+            capi.tune("seq_moe_tc", 1)
+        out[tc, moe_tc] = step_all(m, tokens, [410])
+        rows_within(out[tc, moe_tc], logits, BF16_TOL)
+        m.release()
+        rows_within(step_all(m, tokens, [150, 33, 227]), logits, BF16_TOL)
+        m.close()
+    close(out[2, 1], out[2, 0], 1e-3)
+    rows_within(out[1, 1], out[2, 0], BF16_TOL / 4)
+
+
 def test_forward_steps_use_the_graph_and_match(case):
     cfg, W, tokens, logits, _ = case
     m = on_gpu(cfg, W, capi.PRECISION_F32, chunk=16)

@@ -453,7 +453,6 @@ void destroy(SeqModel* sm) {
 		for (TcWeight* t : {&L.t_in, &L.t_o, &L.t_gu, &L.t_down}) tc_weight_free(t);
 		moe_free(&L.moe);
 	}
-	if (m->moe.h_off) cudaFreeHost(m->moe.h_off);
 	delete m;
 }
 

@@ -489,7 +489,6 @@ void destroy(SeqModel* sm) {
 		for (TcWeight* t : {&L.t_in, &L.t_o, &L.t_uq, &L.t_up, &L.t_down}) tc_weight_free(t);
 		moe_free(&L.moe);
 	}
-	if (m->moe.h_off) cudaFreeHost(m->moe.h_off);
 	delete m;
 }
 

@@ -605,7 +605,6 @@ void destroy(SeqModel* sm) {
 		for (TcWeight* t : {&L.t_in, &L.t_o, &L.t_up, &L.t_down}) tc_weight_free(t);
 		moe_free(&L.moe);
 	}
-	if (m->moe.h_off) cudaFreeHost(m->moe.h_off);
 	delete m;
 }
 

@@ -33,6 +33,7 @@
 
 #include <algorithm>
 
+#include "act_ops.cuh"
 #include "common.cuh"
 
 namespace xalm {
@@ -57,7 +58,6 @@ __device__ __forceinline__ void ld8(const __nv_bfloat16* p, float* o) {
 	o[4] = __uint_as_float(r.z << 16); o[5] = __uint_as_float(r.z & 0xffff0000u);
 	o[6] = __uint_as_float(r.w << 16); o[7] = __uint_as_float(r.w & 0xffff0000u);
 }
-__device__ __forceinline__ float sigmoidf_(float x) { return 1.f / (1.f + expf(-x)); }
 
 // block-wide sum; every thread gets the result.  `red` holds 33 floats of shared memory.
 __device__ __forceinline__ float block_sum(float v, float* red) {
@@ -252,8 +252,6 @@ static __global__ void layer_norm_kernel(const float* __restrict__ x, int ldx, c
 
 // ---- fused epilogues of the row products -------------------------------------------------------------------------------------
 enum { EPI_STORE = 0, EPI_SPLIT_KV = 1, EPI_GLU = 2, EPI_HC = 3, EPI_ACT = 4 };
-enum { GLU_CLAMPED = 0, GLU_SILU = 1, GLU_GELU_TANH = 2 };
-enum { ACT_NONE = 0, ACT_RELU_SQUARED = 1, ACT_SIGMOID = 2, ACT_SILU = 3, ACT_GELU_TANH = 4, ACT_SIGMOID_POW = 5 };
 struct RowsEpi {
 	int kind = EPI_STORE;
 	float* out = nullptr; // STORE / SPLIT_KV / ACT: (T, ldo); GLU: (T, ldo) with ldo = N / 2
@@ -298,28 +296,6 @@ struct RowsEpi {
 	const float* hout = nullptr;
 	const float* scale = nullptr; // layer scale (NULL: none)
 };
-
-__device__ __forceinline__ float glu_clamped(float g, float u, float limit, float alpha) {
-	g = fminf(g, limit);
-	u = fminf(fmaxf(u, -limit), limit);
-	return g * sigmoidf_(alpha * g) * (u + 1.f);
-}
-
-__device__ __forceinline__ float gelu_tanhf_(float z) { return 0.5f * z * (1.f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z))); }
-__device__ __forceinline__ float log_sigmoidf_(float z) { return fminf(z, 0.f) - log1pf(expf(-fabsf(z))); }
-__device__ __forceinline__ float act_apply(int act, float v, float p = 1.f) {
-	if (act == ACT_RELU_SQUARED) { v = fmaxf(v, 0.f); return v * v; }
-	if (act == ACT_SIGMOID) return sigmoidf_(v);
-	if (act == ACT_SILU) return v * sigmoidf_(v);
-	if (act == ACT_GELU_TANH) return gelu_tanhf_(v);
-	if (act == ACT_SIGMOID_POW) return expf(p * log_sigmoidf_(v));
-	return v;
-}
-__device__ __forceinline__ float glu_apply(int act, float g, float u, float limit, float alpha) {
-	if (act == GLU_SILU) return g * sigmoidf_(g) * u;
-	if (act == GLU_GELU_TANH) return gelu_tanhf_(g) * u;
-	return glu_clamped(g, u, limit, alpha);
-}
 
 __device__ __forceinline__ void hc_write(const RowsEpi& e, int row, int col, int width, float v) {
 	const float y = e.scale ? e.scale[col] * v : v;

@@ -197,6 +197,7 @@ struct MoeSortArgs {
 	int* off;     // (E + 1) first place of every expert in `sorted`, or NULL
 	int* inv;     // (T * top) place of every pair in `sorted`, or NULL
 	int n_tiled;  // experts [n_tiled, E) get no tiles (they have no matrices); 0: every expert does
+	int tile_rows; // most rows of a tile; 0: MOE_TM
 };
 // one CTA; shared memory: 2 E + 1 ints
 static __global__ void moe_sort_kernel(MoeSortArgs a) {
@@ -210,12 +211,13 @@ static __global__ void moe_sort_kernel(MoeSortArgs a) {
 	__syncthreads();
 	if (tid == 0) {
 		int at = 0, nt = 0;
+		const int tm = a.tile_rows > 0 ? a.tile_rows : MOE_TM;
 		for (int e = 0; e < a.E; e++) {
 			off[e] = at;
-			for (int r = 0; r < cnt[e] && (a.n_tiled <= 0 || e < a.n_tiled); r += MOE_TM) {
+			for (int r = 0; r < cnt[e] && (a.n_tiled <= 0 || e < a.n_tiled); r += tm) {
 				a.tiles[3 * nt] = e;
 				a.tiles[3 * nt + 1] = at + r;
-				a.tiles[3 * nt + 2] = min(MOE_TM, cnt[e] - r);
+				a.tiles[3 * nt + 2] = min(tm, cnt[e] - r);
 				nt++;
 			}
 			at += cnt[e];
@@ -233,16 +235,6 @@ static __global__ void moe_sort_kernel(MoeSortArgs a) {
 	}
 	if (a.off)
 		for (int e = tid; e <= a.E; e += nth) a.off[e] = off[e];
-}
-
-// rows of the pairs in sorted order, one after the other: dst[place] = src[sorted[place] / div] (the tensor-core products want each expert's rows
-// contiguous)
-static __global__ void moe_gather_kernel(const float* __restrict__ src, int lds, int div, const int* __restrict__ sorted, const SeqStep* step, int top, int width,
-                                         float* __restrict__ dst) {
-	const int place = blockIdx.x;
-	if (place >= step->n * top) return;
-	const float* row = src + (size_t) (sorted[place] / div) * lds;
-	for (int c = threadIdx.x; c < width; c += blockDim.x) dst[(size_t) place * width + c] = row[c];
 }
 
 struct MoeGemmArgs {

@@ -41,6 +41,7 @@
 
 #include "matvec.cuh"
 #include "frag_layout.cuh"
+#include "act_ops.cuh"
 #include "prefill.h"
 
 namespace xalm {
@@ -381,7 +382,7 @@ __device__ __forceinline__ void tmem_ld8(uint32_t taddr, float (&v)[8]) {
 //   warps 2-5 epilogue: tcgen05.ld the 128 x 256 fp32 accumulator (one TMEM lane quadrant per warp) and apply the
 //             fused epilogue, while the MMA warp already fills the OTHER accumulator buffer (2 x 256 of the 512 columns)
 // ------------------------------------------------------------------------------------------------------------------
-enum { GEPI_STORE = 0, GEPI_RESID = 1, GEPI_GLU = 2, GEPI_QKV = 3 };
+enum { GEPI_STORE = 0, GEPI_RESID = 1, GEPI_GLU = 2, GEPI_QKV = 3, GEPI_ACT = 4 /* grouped launches */ };
 
 struct GemmArgs {
 	const uint8_t* a_hi;
@@ -413,6 +414,11 @@ struct GemmArgs {
 	// GLU
 	ATiles o;
 	int act;
+	// grouped launches: row tiles (matrix, first row, rows) instead of MT blocks of one matrix; see TcGroup
+	const int* gtiles;
+	const int* gn_tiles;
+	const uint8_t* const* gb;
+	TcAct gact;
 };
 
 constexpr int GEMM_THREADS = 192;
@@ -425,7 +431,8 @@ struct GemmCfg {
 	static constexpr size_t SMEM = (size_t) NS * STAGE + 1024 /* alignment slack */ + 256 /* barriers */;
 };
 
-template <int NA, int NB>
+// GROUPED: M tiles come from a list, each with a matrix of its own
+template <int NA, int NB, bool GROUPED = false>
 __global__ void __launch_bounds__(GEMM_THREADS, 1) gemm_tc_kernel(const GemmArgs g) {
 	using Cfg = GemmCfg<NA, NB>;
 	constexpr int NS = Cfg::NS;
@@ -457,17 +464,18 @@ __global__ void __launch_bounds__(GEMM_THREADS, 1) gemm_tc_kernel(const GemmArgs
 	tc_fence_after();
 	const uint32_t tmem_base = *reinterpret_cast<volatile uint32_t*>(tmem_slot);
 
-	const int n_tiles = g.MT * g.NT;
+	const int MT = GROUPED ? *g.gn_tiles : g.MT;
+	const int n_tiles = MT * g.NT;
 	const int KT = g.KT;
 
 	if (warp == 0) {
 		if (lane == 0) {
 			int slot = 0, phase = 0;
 			for (int tile = blockIdx.x; tile < n_tiles; tile += gridDim.x) {
-				const int mt = g.mt0 + tile % g.MT, nt = tile / g.MT;
+				const int mt = g.mt0 + tile % MT, nt = tile / MT;
 				const uint8_t* ah = g.a_hi + (size_t) mt * KT * A_TILE_BYTES;
 				const uint8_t* al = NA == 2 ? g.a_lo + (size_t) mt * KT * A_TILE_BYTES : nullptr;
-				const uint8_t* bt = g.b + (size_t) nt * KT * B_TILE_BYTES;
+				const uint8_t* bt = (GROUPED ? g.gb[g.gtiles[3 * mt]] : g.b) + (size_t) nt * KT * B_TILE_BYTES;
 				const uint8_t* bl = NB == 2 ? g.b_lo + (size_t) nt * KT * B_TILE_BYTES : nullptr;
 				for (int kt = 0; kt < KT; kt++) {
 					mb_wait(&empty[slot], phase ^ 1);
@@ -517,13 +525,33 @@ __global__ void __launch_bounds__(GEMM_THREADS, 1) gemm_tc_kernel(const GemmArgs
 		const int quad = warp & 3; // TMEM lanes [32*quad, 32*quad+32) are the ones this warp may read
 		int acc = 0, acc_phase = 0;
 		for (int tile = blockIdx.x; tile < n_tiles; tile += gridDim.x) {
-			const int mt = g.mt0 + tile % g.MT, nt = tile / g.MT;
+			const int mt = g.mt0 + tile % MT, nt = tile / MT;
 			mb_wait(&tfull[acc], acc_phase);
 			tc_fence_after();
 			const int m = mt * GB_M + quad * 32 + lane;
-			const bool mrow = m < g.M;
+			const bool mrow = GROUPED ? quad * 32 + lane < g.gtiles[3 * mt + 2] : m < g.M;
 			const uint32_t taddr = tmem_base + ((uint32_t) (quad * 32) << 16) + (uint32_t) acc * GB_N;
-			if (g.epi == GEPI_GLU) {
+			if (GROUPED && g.epi == GEPI_ACT) {
+				for (int c = 0; c < GB_N; c += 16) {
+					float v[16];
+					tmem_ld16(taddr + c, v);
+					const int n0 = nt * GB_N + c;
+					if (!mrow || n0 >= g.N) continue;
+					float h[8];
+					if (g.gact.glu) { // gate and up columns alternate: 16 columns are 8 values
+#pragma unroll
+						for (int i = 0; i < 8; i++) h[i] = mix::glu_apply(g.gact.act, v[2 * i], v[2 * i + 1], g.gact.limit, g.gact.alpha);
+						store_a8(g.o, m, n0 / 2, h);
+					} else {
+#pragma unroll
+						for (int half = 0; half < 2; half++) {
+#pragma unroll
+							for (int i = 0; i < 8; i++) h[i] = mix::act_apply(g.gact.act, v[8 * half + i]);
+							store_a8(g.o, m, n0 + 8 * half, h);
+						}
+					}
+				}
+			} else if (g.epi == GEPI_GLU) {
 				for (int c = 0; c < GB_N / 2; c += 8) {
 					float gt[8], up[8];
 					tmem_ld8(taddr + c, gt);
@@ -617,7 +645,7 @@ __global__ void __launch_bounds__(GEMM_THREADS, 1) gemm_tc_kernel(const GemmArgs
 					tmem_ld32(taddr + c, v);
 					const int n0 = nt * GB_N + c;
 					if (!mrow || n0 >= g.N) continue;
-					float* o = g.out + (size_t) (m - g.out_row0) * g.ldo + n0;
+					float* o = g.out + (size_t) (GROUPED ? g.gtiles[3 * mt + 1] + quad * 32 + lane : m - g.out_row0) * g.ldo + n0;
 #pragma unroll
 					for (int i = 0; i < 32; i += 4) {
 						if (n0 + i >= g.N) break;
@@ -1378,14 +1406,14 @@ const float* prefill_logits_dev(const PrefillScratch* s, int* rows) {
 	return s ? reinterpret_cast<const float*>(s->logits.p) : nullptr;
 }
 
-template <int NA, int NB>
+template <int NA, int NB, bool GROUPED = false>
 static int launch_gemm_inst(const GemmArgs& g, int grid, cudaStream_t s) {
 	static bool attr = false;
 	if (!attr) {
-		XALM_CUDA_CHECK(cudaFuncSetAttribute(gemm_tc_kernel<NA, NB>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int) GemmCfg<NA, NB>::SMEM));
+		XALM_CUDA_CHECK(cudaFuncSetAttribute(gemm_tc_kernel<NA, NB, GROUPED>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int) GemmCfg<NA, NB>::SMEM));
 		attr = true;
 	}
-	gemm_tc_kernel<NA, NB><<<grid, GEMM_THREADS, GemmCfg<NA, NB>::SMEM, s>>>(g);
+	gemm_tc_kernel<NA, NB, GROUPED><<<grid, GEMM_THREADS, GemmCfg<NA, NB>::SMEM, s>>>(g);
 	return XALM_OK;
 }
 static int launch_gemm(const GemmArgs& g, int na, int nb, cudaStream_t s) {
@@ -1787,6 +1815,56 @@ int tc_gemm(const TcWeight& w, const float* a_dev, int T, float* out_dev, int ld
 	g.a_hi = a_hi; g.a_lo = a_lo; g.b = w.hi; g.b_lo = w.lo;
 	g.MT = MT; g.NT = w.NT; g.KT = w.KT; g.M = T; g.N = w.N; g.epi = GEPI_STORE; g.out = out_dev; g.ldo = ldo;
 	return launch_gemm(g, a_lo ? 2 : 1, w.lo ? 2 : 1, s);
+}
+
+// ---- groups of matrices (prefill.h) -----------------------------------------------------------------------------------------------
+// the ordered rows of every row tile as operand tiles; rows beyond a tile's own are left as they are (no valid row's product depends on them)
+__global__ void pack_group_kernel(const float* __restrict__ a, int K, const int* __restrict__ order, int div, const int* __restrict__ tiles,
+                                  const int* __restrict__ n_tiles, ATiles o) {
+	const int k8s = K / 8, per_tile = GB_M * k8s;
+	const size_t total = (size_t) *n_tiles * per_tile;
+	for (size_t i = blockIdx.x * (size_t) blockDim.x + threadIdx.x; i < total; i += (size_t) gridDim.x * blockDim.x) {
+		const int mt = (int) (i / per_tile), in_tile = (int) (i % per_tile), r = in_tile / k8s, k0 = (in_tile % k8s) * 8;
+		if (r >= tiles[3 * mt + 2]) continue;
+		const float4* src = reinterpret_cast<const float4*>(a + (size_t) (order[tiles[3 * mt + 1] + r] / div) * K + k0);
+		const float4 x = src[0], y = src[1];
+		const float v[8] = {x.x, x.y, x.z, x.w, y.x, y.y, y.z, y.w};
+		store_a8(o, mt * GB_M + r, k0, v);
+	}
+}
+int tc_group_pack(const TcGroup& g, const float* a, const int* order, int div, uint8_t* a_hi, uint8_t* a_lo, cudaStream_t s) {
+	static_assert(TC_TILE_ROWS == GB_M, "a row tile is one M tile");
+	if (g.K % GB_K || g.max_tiles <= 0 || div <= 0) return set_error(XALM_ERR_INVALID, "tc_group_pack: K = %d, %d tiles", g.K, g.max_tiles);
+	const ATiles at{a_hi, a_lo, g.K / GB_K};
+	pack_group_kernel<<<std::min(g.max_tiles * (GB_M * (g.K / 8) / 256), sm_count() * 8), 256, 0, s>>>(a, g.K, order, div, g.tiles, g.n_tiles, at);
+	cudaError_t e = cudaGetLastError();
+	if (e != cudaSuccess) return set_error(XALM_ERR_CUDA, "pack_group launch failed: %s", cudaGetErrorString(e));
+	return XALM_OK;
+}
+static int launch_group(const TcGroup& t, const uint8_t* a_hi, const uint8_t* a_lo, GemmArgs g, cudaStream_t s) {
+	if (t.K % GB_K || t.N % 16 || t.max_tiles <= 0) return set_error(XALM_ERR_INVALID, "tc_group_gemm: %d x %d, %d tiles", t.N, t.K, t.max_tiles);
+	g.a_hi = a_hi; g.a_lo = a_lo;
+	g.NT = cdiv(t.N, GB_N); g.KT = t.K / GB_K; g.N = t.N;
+	g.gtiles = t.tiles; g.gn_tiles = t.n_tiles; g.gb = t.b;
+	const int grid = std::min(t.max_tiles * g.NT, sm_count());
+	if (a_lo) XALM_TRY((launch_gemm_inst<2, 1, true>(g, grid, s)));
+	else XALM_TRY((launch_gemm_inst<1, 1, true>(g, grid, s)));
+	cudaError_t e = cudaGetLastError();
+	if (e != cudaSuccess) return set_error(XALM_ERR_CUDA, "grouped gemm_tc launch failed: %s", cudaGetErrorString(e));
+	return XALM_OK;
+}
+int tc_group_gemm_act(const TcGroup& t, const uint8_t* a_hi, const uint8_t* a_lo, const TcAct& act, uint8_t* o_hi, uint8_t* o_lo, cudaStream_t s) {
+	GemmArgs g = {};
+	g.epi = GEPI_ACT;
+	g.gact = act;
+	g.o = ATiles{o_hi, o_lo, (act.glu ? t.N / 2 : t.N) / GB_K};
+	return launch_group(t, a_hi, a_lo, g, s);
+}
+int tc_group_gemm(const TcGroup& t, const uint8_t* a_hi, const uint8_t* a_lo, float* out, int ldo, cudaStream_t s) {
+	GemmArgs g = {};
+	g.epi = GEPI_STORE;
+	g.out = out; g.ldo = ldo;
+	return launch_group(t, a_hi, a_lo, g, s);
 }
 
 } // namespace xalm

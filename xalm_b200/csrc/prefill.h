@@ -69,4 +69,29 @@ size_t tc_a_plane_bytes(int T, int K); // one operand plane of T x K activations
 // Two launches (pack, GEMM) on stream s; nothing is synchronised.
 int tc_gemm(const TcWeight& w, const float* a_dev, int T, float* out_dev, int ldo, uint8_t* a_hi, uint8_t* a_lo, cudaStream_t s);
 
+
+// ---- the same for a group of equally shaped matrices (the experts of a mixture): one launch runs every matrix's own rows -------------------
+// The rows come as a list of row tiles of at most TC_TILE_ROWS rows: tiles[3 i] = which matrix, tiles[3 i + 1] = the tile's first place in
+// the ordered rows, tiles[3 i + 2] = its rows; how many tiles there are is only known on the device.
+constexpr int TC_TILE_ROWS = 128;
+struct TcGroup {
+	const uint8_t* const* b = nullptr; // (device) fp16 B tiles of every matrix (TcWeight::hi)
+	int N = 0, K = 0;
+	const int* tiles = nullptr;
+	const int* n_tiles = nullptr;
+	int max_tiles = 0;
+};
+// what happens to a product that is the next one's operand: pairs of neighbouring columns (gate, up) become one value, or each value its own
+struct TcAct {
+	bool glu = false;
+	int act = 0; // GLU_* or ACT_* (act_ops.cuh)
+	float limit = 0.f, alpha = 0.f;
+};
+// operand tiles of the ordered rows: row `place` is row order[place] / div of `a` (K floats each)
+int tc_group_pack(const TcGroup& g, const float* a, const int* order, int div, uint8_t* a_hi, uint8_t* a_lo, cudaStream_t s);
+// operand tiles -> act -> operand tiles of the next product (K: N / 2 for a GLU, else N)
+int tc_group_gemm_act(const TcGroup& g, const uint8_t* a_hi, const uint8_t* a_lo, const TcAct& act, uint8_t* o_hi, uint8_t* o_lo, cudaStream_t s);
+// operand tiles -> fp32 rows at their places in the order
+int tc_group_gemm(const TcGroup& g, const uint8_t* a_hi, const uint8_t* a_lo, float* out, int ldo, cudaStream_t s);
+
 } // namespace xalm

@@ -2,8 +2,8 @@
 // and the kernels of moe_ops.cuh in order.
 //
 //   router -> [steps of a few tokens: one matvec per (token, slot) pair] or [sort by expert -> tiled fp32 products] or, for long passes of the
-//   16-bit mode, [sort -> gather -> every expert's rows through the tcgen05 GEMM on that expert's resident fp16 tiles]; the caller then joins
-//   each token's expert rows (moe_combine, with whatever else its layer adds there).
+//   16-bit mode, [sort -> rows packed in expert order -> grouped tcgen05 GEMM with the activation fused -> grouped tcgen05 GEMM] on the experts'
+//   resident fp16 tiles; the caller then joins each token's expert rows (moe_combine, with whatever else its layer adds there).
 //
 // A family says what differs between designs: how scores become choices and weights (MoeRouteArgs), the activation between an expert's two
 // products (RowsEpi), how many of the router's outputs are identity experts.
@@ -24,15 +24,17 @@ struct MoeWeights {
 	float* correction = nullptr; // (E + identity) or NULL
 	WMat m_up, m_down;
 	std::vector<TcWeight> t_up, t_down; // per expert, when long passes run on the tensor cores
+	const uint8_t **b_up = nullptr, **b_down = nullptr; // (device) their tiles
 	bool on_tc(const SeqModel* m, int n) const { return m->use_tc && !t_up.empty() && n > 1 && n >= m->tc_min_rows; }
 };
 
 struct MoeBuffers { // of one pass, sized for the largest mixture of the model
 	size_t max_pairs = 0, max_hid = 0;
-	int max_tiles = 1, max_outputs = 1;
-	bool tc = false;
-	int *idx = nullptr, *sorted = nullptr, *tiles = nullptr, *ntiles = nullptr, *off = nullptr, *inv = nullptr, *h_off = nullptr;
-	float *wgt = nullptr, *hid = nullptr, *out = nullptr, *x = nullptr;
+	int max_tiles = 1;
+	size_t a_bytes = 0, h_bytes = 0; // operand planes of the tensor-core products: the mixture's input rows in expert order, the hidden rows
+	int *idx = nullptr, *sorted = nullptr, *tiles = nullptr, *ntiles = nullptr, *inv = nullptr;
+	float *wgt = nullptr, *hid = nullptr, *out = nullptr;
+	uint8_t *a_hi = nullptr, *a_lo = nullptr, *hid_hi = nullptr, *hid_lo = nullptr;
 };
 
 // tensors of `E` experts under prefix p ("<p>e0." ...): gate (when gated), up, down
@@ -63,9 +65,11 @@ int moe_upload(SeqModel* m, const std::string& p, bool gated, MoeWeights* L, Moe
 	b->max_pairs = std::max(b->max_pairs, pairs);
 	b->max_hid = std::max(b->max_hid, pairs * L->ff);
 	b->max_tiles = std::max(b->max_tiles, moe_max_tiles((int) pairs, L->E));
-	b->max_outputs = std::max(b->max_outputs, L->E + L->identity);
 	return XALM_OK;
 }
+
+// row tiles of the grouped GEMM over `pairs` rows: every expert may end with a partly filled one
+inline int moe_tc_tiles(int pairs, int E) { return pairs / TC_TILE_ROWS + std::min(E, pairs); }
 
 // a mixture whose expert shapes the GEMM takes keeps fp16 tiles per expert for its long passes
 int moe_tc_register(SeqModel* m, MoeWeights* L, MoeBuffers* b) {
@@ -82,7 +86,15 @@ int moe_tc_register(SeqModel* m, MoeWeights* L, MoeBuffers* b) {
 		XALM_TRY(tc_register(m, up, &L->t_up[(size_t) e]));
 		XALM_TRY(tc_register(m, dn, &L->t_down[(size_t) e]));
 	}
-	b->tc = true;
+	std::vector<const uint8_t*> up((size_t) L->E), dn((size_t) L->E);
+	for (int e = 0; e < L->E; e++) { up[(size_t) e] = L->t_up[(size_t) e].hi; dn[(size_t) e] = L->t_down[(size_t) e].hi; }
+	XALM_TRY(dev_alloc(m, &L->b_up, up.size()));
+	XALM_TRY(dev_alloc(m, &L->b_down, dn.size()));
+	XALM_CUDA_CHECK(cudaMemcpy(L->b_up, up.data(), up.size() * sizeof up[0], cudaMemcpyHostToDevice));
+	XALM_CUDA_CHECK(cudaMemcpy(L->b_down, dn.data(), dn.size() * sizeof dn[0], cudaMemcpyHostToDevice));
+	const int rows = moe_tc_tiles(m->chunk * L->top, L->E) * TC_TILE_ROWS;
+	b->a_bytes = std::max(b->a_bytes, tc_a_plane_bytes(rows, W));
+	b->h_bytes = std::max(b->h_bytes, tc_a_plane_bytes(rows, L->ff));
 	return XALM_OK;
 }
 
@@ -96,11 +108,14 @@ int moe_alloc(SeqModel* m, MoeBuffers* b) {
 	XALM_TRY(dev_alloc(m, &b->ntiles, 1, true));
 	XALM_TRY(dev_alloc(m, &b->hid, b->max_hid));
 	XALM_TRY(dev_alloc(m, &b->out, b->max_pairs * W));
-	if (b->tc) {
-		XALM_TRY(dev_alloc(m, &b->off, (size_t) b->max_outputs + 1, true));
+	if (b->a_bytes) {
 		XALM_TRY(dev_alloc(m, &b->inv, b->max_pairs, true));
-		XALM_TRY(dev_alloc(m, &b->x, b->max_pairs * W));
-		XALM_CUDA_CHECK(cudaMallocHost(&b->h_off, ((size_t) b->max_outputs + 1) * 4));
+		XALM_TRY(dev_alloc(m, &b->a_hi, b->a_bytes, true));
+		XALM_TRY(dev_alloc(m, &b->hid_hi, b->h_bytes, true));
+		if (tune("seq_tc") >= 2) {
+			XALM_TRY(dev_alloc(m, &b->a_lo, b->a_bytes, true));
+			XALM_TRY(dev_alloc(m, &b->hid_lo, b->h_bytes, true));
+		}
 	}
 	return XALM_OK;
 }
@@ -123,27 +138,25 @@ int moe_experts(SeqModel* m, const MoeWeights& L, const MoeBuffers& b, const flo
 	(*nl)++;
 	const bool on_tc = L.on_tc(m, n);
 	if (on_tc || n * L.top > MOE_MATVEC_PAIRS) { // steps of a few tokens need no tile list
-		MoeSortArgs so = {b.idx, L.top, total, m->d_step, b.sorted, b.tiles, b.ntiles, b.off, b.inv, L.E};
+		MoeSortArgs so = {b.idx, L.top, total, m->d_step, b.sorted, b.tiles, b.ntiles, nullptr, b.inv, L.E, on_tc ? TC_TILE_ROWS : 0};
 		XALM_TRY(launch_moe_sort(so, s));
 		(*nl)++;
 	}
 	act.ldo = L.ff;
 	if (on_tc) {
-		// Each expert's rows, gathered one after the other, go through the GEMM.  How many rows each expert got is read back first (one small copy
-		// and a wait per mixture layer and pass).
-		XALM_CUDA_CHECK(cudaMemcpyAsync(b.h_off, b.off, (size_t) (total + 1) * 4, cudaMemcpyDeviceToHost, s));
-		moe_gather_kernel<<<n * L.top, 256, 0, s>>>(h, W, L.top, b.sorted, m->d_step, L.top, W, b.x);
-		XALM_SEQ_LAUNCH_CHECK("moe_gather");
-		XALM_CUDA_CHECK(cudaStreamSynchronize(s));
-		for (int e = 0; e < L.E; e++) {
-			const int at = b.h_off[e], cnt = b.h_off[e + 1] - at;
-			if (cnt <= 0) continue;
-			XALM_TRY(tc_gemm(L.t_up[(size_t) e], b.x + (size_t) at * W, cnt, m->tc_out, L.up_rows, m->a_hi, m->a_lo, s));
-			act.out = b.hid + (size_t) at * L.ff;
-			XALM_TRY(launch_rows_epilogue(m->tc_out, L.up_rows, cnt, L.up_rows, act, s));
-			XALM_TRY(tc_gemm(L.t_down[(size_t) e], b.hid + (size_t) at * L.ff, cnt, b.out + (size_t) at * W, W, m->a_hi, m->a_lo, s));
-			*nl += 5;
-		}
+		TcGroup up, dn;
+		up.b = L.b_up; up.N = L.up_rows; up.K = W;
+		up.tiles = b.tiles; up.n_tiles = b.ntiles; up.max_tiles = moe_tc_tiles(n * L.top, L.E);
+		dn = up;
+		dn.b = L.b_down; dn.N = W; dn.K = L.ff;
+		TcAct ta;
+		ta.glu = act.kind == EPI_GLU;
+		ta.act = ta.glu ? act.glu_act : act.act;
+		ta.limit = act.limit; ta.alpha = act.alpha;
+		XALM_TRY(tc_group_pack(up, h, b.sorted, L.top, b.a_hi, b.a_lo, s));
+		XALM_TRY(tc_group_gemm_act(up, b.a_hi, b.a_lo, ta, b.hid_hi, b.hid_lo, s));
+		XALM_TRY(tc_group_gemm(dn, b.hid_hi, b.hid_lo, b.out, W, s));
+		*nl += 3;
 	} else {
 		MoeGemmArgs ga = {};
 		ga.A = h; ga.lda = W; ga.a_div = L.top; ga.W = L.w_up; ga.N = L.up_rows; ga.K = W;
