@@ -1029,7 +1029,6 @@ struct AttnTcArgs {
 	const uint8_t* vt;   // V^T tiles
 	ATiles o;            // xb2
 	int T, pos0, n_heads, n_kv_heads, n_qb, n_kb_total;
-	int dbg; // timing knock-outs (XALM_ATTN_DBG, results are then meaningless): 1 = no QK MMAs, 2 = no PV MMAs, 4 = no softmax math / P stores
 };
 
 // cache rows -> K tiles and V^T tiles.  grid (64-key blocks, kv heads), 256 threads.
@@ -1154,9 +1153,7 @@ __global__ void __launch_bounds__(ATT_THREADS, 1) attn_tc_kernel(const AttnTcArg
 		__syncwarp();
 	} else if (warp == 1) {
 		// The whole warp runs the control flow (barrier waits included) and ONE elected lane issues the MMAs and commits inside a
-		// warp-uniform branch.  With the loop under `if (lane == 0)` instead, ncu showed ~210 instructions per 64-key block on this
-		// single thread (ELECT / PLOP3 / R2UR around every UTCHMMA) — the MMA issuer, not the tensor pipe (28 % active) or the
-		// softmax warps, was setting the pace.
+		// warp-uniform branch; operand descriptors are built once, so that the issuing thread does little else per block.
 		constexpr uint32_t idesc_s = instr_desc_f16(128, ATT_BKV); // S = Q K^T: 128 rows x 64 keys
 		constexpr uint32_t idesc_o = instr_desc_f16(128, 128);     // O += P V: 128 rows x 128 hd
 		const uint32_t q_s = s_u32(sQ), p_s = s_u32(sP), k_s = s_u32(sK), v_s = s_u32(sV);
@@ -1186,7 +1183,7 @@ __global__ void __launch_bounds__(ATT_THREADS, 1) attn_tc_kernel(const AttnTcArg
 					for (int t = 0; t < 2; t++) // hd halves
 #pragma unroll
 						for (int k = 0; k < 4; k++)
-							if (!(a.dbg & 1)) umma_f16(d, qd[p * 2 + t] + 2 * k, (t ? kd1 : kd0) + 2 * k, idesc_s, (uint32_t) ((p | t | k) != 0));
+							umma_f16(d, qd[p * 2 + t] + 2 * k, (t ? kd1 : kd0) + 2 * k, idesc_s, (uint32_t) ((p | t | k) != 0));
 				umma_commit(&k_empty[slot]);
 				umma_commit(&s_full[b]);
 			}
@@ -1210,7 +1207,7 @@ __global__ void __launch_bounds__(ATT_THREADS, 1) attn_tc_kernel(const AttnTcArg
 					const uint64_t pdd = b ? pd[NP + p] : pd[p];
 #pragma unroll
 					for (int k = 0; k < 4; k++)
-						if (!(a.dbg & 2)) umma_f16(TM_O, pdd + 2 * k, vdd + 2 * k, idesc_o, (uint32_t) ((j | p | k) != 0)); // O accumulates over all blocks
+						umma_f16(TM_O, pdd + 2 * k, vdd + 2 * k, idesc_o, (uint32_t) ((j | p | k) != 0)); // O accumulates over all blocks
 				}
 				umma_commit(&v_empty[slot]);
 				umma_commit(&o_full[b]);
@@ -1279,7 +1276,7 @@ __global__ void __launch_bounds__(ATT_THREADS, 1) attn_tc_kernel(const AttnTcArg
 			uint8_t* pt = sP + (size_t) (b * NP) * Cfg::P_TILE;
 			float rs = 0.f;
 #pragma unroll
-			for (int g8 = 0; g8 < ((a.dbg & 4) ? 0 : ATT_BKV / 8); g8++) { // 8 keys = one 16-byte chunk
+			for (int g8 = 0; g8 < ATT_BKV / 8; g8++) { // 8 keys = one 16-byte chunk
 				__half2 hh[4], ll[4];
 #pragma unroll
 				for (int i = 0; i < 4; i++) {
@@ -1641,8 +1638,7 @@ int prefill_run(const PrefillModel& pm, PrefillScratch** scratch, const int* tok
 		if (attn_tc) {
 			if (!tiles_from_epilogue)
 				retile_kv_kernel<<<dim3(2 * n_kb_total, c.n_kv_heads), 256, 0, s>>>(P.k_cache, P.v_cache, pm.kv_dim, pos0 + T, n_kb_total, sc.kt.p, sc.vt.p);
-			AttnTcArgs at = {sc.qt_hi.p, precise ? sc.qt_lo.p : nullptr, sc.kt.p, sc.vt.p, xb2, T, pos0, c.n_heads, c.n_kv_heads, n_qb, n_kb_total,
-			                 getenv("XALM_ATTN_DBG") ? atoi(getenv("XALM_ATTN_DBG")) : 0};
+			AttnTcArgs at = {sc.qt_hi.p, precise ? sc.qt_lo.p : nullptr, sc.kt.p, sc.vt.p, xb2, T, pos0, c.n_heads, c.n_kv_heads, n_qb, n_kb_total};
 			XALM_TRY(precise ? launch_attn_tc<true>(at, s) : launch_attn_tc<false>(at, s));
 			launches++;
 		} else {
