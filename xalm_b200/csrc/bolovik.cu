@@ -86,7 +86,7 @@ typedef BolovikModel Bv;
 // ---- config.json ------------------------------------------------------------------------------------------------------------------
 // rotary frequencies f_i = base^(-2i/dims), rescaled by wavelength l = 2 pi / f: kept where l < original / high, divided by `factor` where
 // l > original / low, blended linearly in (original / l) between the two
-std::vector<float> rotary_frequencies(const xjson::Value& rot, int dims) {
+std::vector<float> scaled_frequencies(const xjson::Value& rot, int dims) {
 	const double base = getf(rot, "base");
 	const xjson::Value* sc = rot.find("scaling");
 	const bool scaled = sc && sc->kind == xjson::Value::Obj;
@@ -151,7 +151,7 @@ int parse_config(SeqModel* sm, const char* json) {
 				if (const xjson::Value* rt = mx.find("rot"); rt && rt->kind == xjson::Value::Obj) {
 					L.rot_dims = geti(*rt, "dims");
 					if (L.rot_dims < 0 || L.rot_dims > d || L.rot_dims % 2) return set_error(XALM_ERR_INVALID, "config: layer %zu: %d rotary dimensions in a head of %d", li, L.rot_dims, d);
-					if (L.rot_dims) L.freq_host = rotary_frequencies(*rt, L.rot_dims);
+					if (L.rot_dims) L.freq_host = scaled_frequencies(*rt, L.rot_dims);
 				}
 				expect(m, p + "mix.q", {H * d, W}, true);
 				expect(m, p + "mix.q.b", {H * d}, false, false);

@@ -14,7 +14,7 @@
 // x <- x + mixer(rmsnorm(x) w1), x <- x + ff(rmsnorm(x) w2); the embedding row is scaled; logits = cap * tanh(head . rmsnorm(x) / cap).
 //
 // The step function, graph replay of one-token steps, uploads, release and the C entry points are the shared sequence engine's
-// (seq_family.cuh).  Per pass and layer here:
+// (seq_family.cuh), the latent mixers' kernels in order are seq_latent.cuh's.  Per pass and layer here:
 //     latent attention: norm -> rows product [dq | dkv | gate] -> latent_post (latent norms, rotated key, cache row) -> rows product [uq]
 //                       -> batched per-head product with uk^T (queries into the latent) + rope_heads (rotated query part) -> swa_attn /
 //                       swa_tile with ONE key/value head reading the cache rows in place -> batched per-head product with uv (gate fused)
@@ -33,7 +33,7 @@
 // the tcgen05 GEMM (fp16 operands, fp32 accumulation); XALM_PRECISION_F32 widens both and uses the fp32 FMA kernels only.
 #include "seq_family.cuh"
 
-#include "latent_ops.cuh"
+#include "seq_latent.cuh"
 #include "seq_moe.cuh"
 
 namespace xalm {
@@ -48,23 +48,17 @@ enum { FF_NONE = 0, FF_DENSE = 1, FF_MOE = 2 };
 struct Layer {
 	int mixer = MIX_LATENT, ff_kind = FF_NONE;
 	int H = 0, d = 0, dv = 0;
-	// latent attention: r rotated entries per head, R / Rq latent sizes of keys+values / queries
-	int r = 0, R = 0, Rq = 0, kv_from = -1;
-	float scale = 1.f;
-	float *dq_norm = nullptr, *dkv_norm = nullptr;
-	void* cache = nullptr; // (max_tokens, cache_ld): this layer's rows, or the rows of the layer it reads
-	int cache_ld = 0;
-	void *w_uq = nullptr, *w_ukT = nullptr, *w_uv = nullptr;
-	WMat m_uq;
-	TcWeight t_uq;
+	// latent attention
+	LatentWeights lat;
+	int kv_from = -1;
+	LatentCache cache; // this layer's rows, or the rows of the layer it reads
 	// retention
 	int rot_dims = 0;
 	std::vector<float> decay_host;
 	float *decay = nullptr, *state = nullptr;
-	// both
 	std::vector<float> freq_host;
 	float* freq = nullptr;
-	int off_a = 0, off_b = 0, off_g = 0, n_in = 0; // columns of the stacked input projection: [dq | dkv | g] or [q | k | v | g]
+	int off_a = 0, off_b = 0, off_g = 0, n_in = 0; // columns of the stacked input projection [q | k | v | g]
 	// feed-forward
 	int ff = 0; // dense
 	MoeWeights moe;
@@ -79,20 +73,13 @@ struct DuletarModel : SeqModel {
 	float embed_scale = 1.f, logit_cap = 0.f;
 	std::vector<Layer> layers;
 	// one pass
-	float *x = nullptr, *hn = nullptr, *proj = nullptr, *cq = nullptr, *q = nullptr, *qabs = nullptr, *olat = nullptr, *att = nullptr, *ffh = nullptr;
+	float *x = nullptr, *hn = nullptr, *proj = nullptr, *att = nullptr, *ffh = nullptr;
 	int proj_ld = 4;
-	float *part_o = nullptr, *part_ml = nullptr;
-	unsigned* tickets = nullptr;
-	int part_cap = 0;
+	LatentBuffers lat;
+	AttnParts parts;
 	MoeBuffers moe;
 };
 typedef DuletarModel Du;
-
-std::vector<float> rotary_frequencies(double base, int dims) { // f_i = base^(-2i/dims)
-	std::vector<float> f((size_t) dims / 2);
-	for (int i = 0; i < dims / 2; i++) f[(size_t) i] = (float) pow(base, -2.0 * i / dims);
-	return f;
-}
 
 // ---- config.json ------------------------------------------------------------------------------------------------------------------
 int parse_config(SeqModel* sm, const char* json) {
@@ -142,38 +129,33 @@ int parse_config(SeqModel* sm, const char* json) {
 				expect(m, p + "mix.v", {H * dv, W}, true);
 				expect(m, p + "mix.g", {H * dv, W}, true);
 			} else {
-				L.R = geti(mx, "kv_rank");
-				L.Rq = geti(mx, "q_rank");
-				L.scale = mx.contains("scale") ? (float) getf(mx, "scale") : 1.f / sqrtf((float) d);
+				LatentWeights& A = L.lat;
+				A.H = H; A.d = d; A.dv = dv;
+				A.R = geti(mx, "kv_rank");
+				A.Rq = geti(mx, "q_rank");
+				A.gate = L.mixer == MIX_LATENT_GATED ? LATENT_GATE_COLUMNS : LATENT_GATE_NONE;
+				A.scale = mx.contains("scale") ? (float) getf(mx, "scale") : 1.f / sqrtf((float) d);
 				if (L.mixer == MIX_LATENT) {
-					L.r = mx.contains("rot_dim") ? geti(mx, "rot_dim") : 0;
-					if (L.r < 0 || L.r % 2) return set_error(XALM_ERR_INVALID, "config: layer %zu: rot_dim %d", li, L.r);
-					if (L.r) {
+					A.r = mx.contains("rot_dim") ? geti(mx, "rot_dim") : 0;
+					if (A.r < 0 || A.r % 2) return set_error(XALM_ERR_INVALID, "config: layer %zu: rot_dim %d", li, A.r);
+					if (A.r) {
 						if (!rt) return set_error(XALM_ERR_INVALID, "config: layer %zu: rot_dim without 'rot'", li);
-						const int dims = rt->contains("dims") ? geti(*rt, "dims") : L.r;
-						if (dims != L.r) return set_error(XALM_ERR_INVALID, "config: layer %zu: rot.dims %d differs from rot_dim %d", li, dims, L.r);
-						L.freq_host = rotary_frequencies(getf(*rt, "base"), L.r);
+						const int dims = rt->contains("dims") ? geti(*rt, "dims") : A.r;
+						if (dims != A.r) return set_error(XALM_ERR_INVALID, "config: layer %zu: rot.dims %d differs from rot_dim %d", li, dims, A.r);
+						A.freq_host = rotary_frequencies(getf(*rt, "base"), A.r);
 					}
 				}
-				if (L.R <= 0 || L.Rq <= 0) return set_error(XALM_ERR_INVALID, "config: layer %zu: latent sizes", li);
+				if (A.R <= 0 || A.Rq <= 0) return set_error(XALM_ERR_INVALID, "config: layer %zu: latent sizes", li);
 				if (const xjson::Value* kf = mx.find("kv_from"); kf && kf->kind == xjson::Value::Number) {
 					if (L.mixer != MIX_LATENT_GATED) return set_error(XALM_ERR_UNSUPPORTED, "config: layer %zu: kv_from on a rotary latent attention", li);
 					L.kv_from = (int) kf->num;
 					if (L.kv_from < 0 || L.kv_from >= (int) li) return set_error(XALM_ERR_INVALID, "config: layer %zu: kv_from %d is not an earlier layer", li, L.kv_from);
 					const Layer& J = m->layers[(size_t) L.kv_from];
-					if (J.mixer == MIX_RETENTION || J.kv_from >= 0 || J.R != L.R)
-						return set_error(XALM_ERR_INVALID, "config: layer %zu: layer %d has no latents of %d of its own", li, L.kv_from, L.R);
+					if (J.mixer == MIX_RETENTION || J.kv_from >= 0 || J.lat.R != A.R)
+						return set_error(XALM_ERR_INVALID, "config: layer %zu: layer %d has no latents of %d of its own", li, L.kv_from, A.R);
 				}
-				expect(m, p + "mix.dq", {L.Rq, W}, true);
-				expect(m, p + "mix.dq.norm", {L.Rq}, false);
-				expect(m, p + "mix.uq", {H * (d + L.r), L.Rq}, true);
-				if (L.kv_from < 0) {
-					expect(m, p + "mix.dkv", {L.R + L.r, W}, true);
-					expect(m, p + "mix.dkv.norm", {L.R}, false);
-				}
-				expect(m, p + "mix.uk", {H * d, L.R}, true);
-				expect(m, p + "mix.uv", {H * dv, L.R}, true);
-				if (L.mixer == MIX_LATENT_GATED) expect(m, p + "mix.g", {H * dv, W}, true);
+				A.own_cache = L.kv_from < 0;
+				latent_expect(m, p + "mix.", A);
 			}
 			expect(m, p + "mix.o", {W, H * dv}, true);
 			const xjson::Value* mlp = lv.find("mlp");
@@ -226,56 +208,6 @@ RowsEpi residual_epi(Du* m) { // x <- x + product: the single-stream case of the
 	return e;
 }
 
-int enqueue_latent(Du* m, const Layer& L, int n, int* nl) {
-	cudaStream_t s = m->stream;
-	const int H = L.H, d = L.d, r = L.r, dv = L.dv, R = L.R, Rq = L.Rq;
-	const bool f32 = m->precision == XALM_PRECISION_F32;
-	LatentPostArgs pa = {};
-	pa.proj = m->proj; pa.ld = m->proj_ld;
-	pa.q_off = 0; pa.q_rank = Rq; pa.q_norm = L.dq_norm; pa.cq = m->cq; pa.ldc = Rq;
-	pa.kv_off = L.off_a; pa.kv_rank = L.kv_from < 0 ? R : 0; pa.rot = r; pa.kv_norm = L.dkv_norm; pa.freq = L.freq;
-	pa.eps = m->eps; pa.cache = L.cache; pa.cache_f32 = f32; pa.ring = m->max_tokens; pa.step = m->d_step;
-	XALM_TRY(launch_latent_post(pa, n, s));
-	(*nl)++;
-	RowsEpi est;
-	est.kind = EPI_STORE; est.out = m->q; est.ldo = H * (d + r);
-	XALM_TRY(rows_product(m, m->cq, Rq, L.w_uq, &L.t_uq, n, H * (d + r), Rq, est, nl));
-	// queries into the latent, head by head: qabs[h] = [uk_h^T q_h | rotated q_h]
-	RowsEpi eb;
-	eb.kind = EPI_STORE; eb.out = m->qabs; eb.ldo = H * (R + r);
-	eb.batch_a = d + r; eb.batch_w = (size_t) R * d; eb.batch_o = R + r;
-	XALM_TRY(launch_rows(m->q, H * (d + r), L.w_ukT, m->w_bf16, n, R, d, eb, s, H));
-	(*nl)++;
-	if (r) {
-		RopeHeadsArgs ra = {};
-		ra.src = m->q; ra.lds = H * (d + r); ra.src_off = d; ra.src_stride = d + r;
-		ra.dst = m->qabs; ra.ldd = H * (R + r); ra.dst_off = R; ra.dst_stride = R + r;
-		ra.heads = H; ra.n = r; ra.rot_half = r / 2; ra.freq = L.freq; ra.step = m->d_step;
-		XALM_TRY(launch_rope_heads(ra, n, s));
-		(*nl)++;
-	}
-	SwaArgs sa = {};
-	sa.q = m->qabs; sa.ldq = H * (R + r); sa.q_off = 0;
-	sa.kc = L.cache; sa.vc = L.cache; sa.ldk = L.cache_ld; sa.ldv = L.cache_ld;
-	sa.ring = m->max_tokens; sa.keep_first = 0;
-	sa.H = H; sa.G = 1; sa.d = R + r; sa.dv = R;
-	sa.window = 0x7fffffff; sa.scale = L.scale;
-	sa.step = m->d_step; sa.out = m->olat;
-	sa.n_splits = 0;
-	sa.part_o = m->part_o; sa.part_ml = m->part_ml; sa.part_cap = m->part_cap; sa.tickets = m->tickets;
-	int swa_launches = 1;
-	XALM_TRY(launch_swa(sa, n, f32, s, &swa_launches));
-	*nl += swa_launches;
-	// values out of the latent, head by head, with the output gate
-	RowsEpi ev;
-	ev.kind = EPI_STORE; ev.out = m->att; ev.ldo = H * dv;
-	ev.batch_a = R; ev.batch_w = (size_t) dv * R; ev.batch_o = dv;
-	if (L.mixer == MIX_LATENT_GATED) { ev.mul = m->proj + L.off_g; ev.ldm = m->proj_ld; ev.mul_act = ACT_SIGMOID; }
-	XALM_TRY(launch_rows(m->olat, H * R, L.w_uv, m->w_bf16, n, dv, R, ev, s, H));
-	(*nl)++;
-	return XALM_OK;
-}
-
 int enqueue_retention(Du* m, const Layer& L, int n, int* nl) {
 	cudaStream_t s = m->stream;
 	const int H = L.H, d = L.d, dv = L.dv;
@@ -325,9 +257,13 @@ int enqueue_pass(SeqModel* sm, int n, int want, int* nl) {
 		(*nl)++;
 		RowsEpi est;
 		est.kind = EPI_STORE; est.out = m->proj; est.ldo = m->proj_ld;
-		XALM_TRY(rows_product(m, m->hn, W, L.w_in, &L.t_in, n, L.n_in, W, est, nl));
-		if (L.mixer == MIX_RETENTION) XALM_TRY(enqueue_retention(m, L, n, nl));
-		else XALM_TRY(enqueue_latent(m, L, n, nl));
+		if (L.mixer == MIX_RETENTION) {
+			XALM_TRY(rows_product(m, m->hn, W, L.w_in, &L.t_in, n, L.n_in, W, est, nl));
+			XALM_TRY(enqueue_retention(m, L, n, nl));
+		} else {
+			XALM_TRY(rows_product(m, m->hn, W, L.lat.w_in, &L.lat.t_in, n, L.lat.n_in, W, est, nl));
+			XALM_TRY(latent_attention(m, L.lat, L.cache, m->lat, m->parts, m->proj, m->proj_ld, m->att, n, nl));
+		}
 		XALM_TRY(rows_product(m, m->att, L.H * L.dv, L.w_o, &L.t_o, n, W, L.H * L.dv, residual_epi(m), nl));
 		if (L.ff_kind != FF_NONE) {
 			XALM_TRY(launch_hc_norm(m->x, 1, hs, nullptr, L.norm2, 0, m->eps, W, m->hn, nullptr, n, s));
@@ -353,28 +289,16 @@ int enqueue_pass(SeqModel* sm, int n, int want, int* nl) {
 }
 
 // ---- device layouts, cache, state, pass buffers ---------------------------------------------------------------------------------------
-// uk (H * d, R) as H matrices (R, d): row j of head h holds column j of that head's rows, so that q_h -> uk_h^T q_h is a rows product
-int upload_transposed_heads(Du* m, const HostTensor* uk, int H, int d, int R, void** dst) {
-	HostTensor t;
-	t.shape = {H * R, d};
-	t.v.resize((size_t) H * R * d);
-	for (int h = 0; h < H; h++)
-		for (int i = 0; i < d; i++)
-			for (int j = 0; j < R; j++) t.v[((size_t) h * R + j) * d + i] = uk->v[((size_t) h * d + i) * R + j];
-	return upload_rows(m, {&t}, d, false, dst, nullptr);
-}
-
 int finalize(SeqModel* sm) {
 	Du* m = static_cast<Du*>(sm);
 	const int W = m->width;
 	const size_t C = (size_t) m->chunk;
 	auto T = [&](const std::string& n) { return tensor_or_null(m, n); };
-	size_t max_in = 4, max_cq = 1, max_q = 1, max_qabs = 1, max_olat = 1, max_att = 1, max_ff = 1, max_h = 1;
-	const size_t kelem = m->precision == XALM_PRECISION_F32 ? 4 : 2;
+	size_t max_in = 4, max_att = 1, max_ff = 1;
 	for (size_t li = 0; li < m->layers.size(); li++) {
 		Layer& L = m->layers[li];
 		const std::string p = "l" + std::to_string(li) + ".";
-		const int H = L.H, d = L.d, dv = L.dv, r = L.r, R = L.R, Rq = L.Rq;
+		const int H = L.H, d = L.d, dv = L.dv;
 		XALM_TRY(upload_vec(m, p + "norm1", &L.norm1));
 		if (!L.freq_host.empty()) XALM_TRY(upload_floats(m, L.freq_host.data(), L.freq_host.size(), &L.freq));
 		if (L.mixer == MIX_RETENTION) {
@@ -386,33 +310,10 @@ int finalize(SeqModel* sm) {
 				return set_error(XALM_ERR_UNSUPPORTED, "layer %zu: a retention state of %d x %d per head", li, d, dv);
 			XALM_TRY(hgrn2_prepare(d, dv));
 		} else {
-			const bool own = L.kv_from < 0;
-			L.off_a = Rq; L.off_g = Rq + (own ? R + r : 0);
-			L.n_in = L.off_g + (L.mixer == MIX_LATENT_GATED ? H * dv : 0);
-			XALM_TRY(upload_rows(m, {T(p + "mix.dq"), own ? T(p + "mix.dkv") : nullptr, L.mixer == MIX_LATENT_GATED ? T(p + "mix.g") : nullptr}, W, false, &L.w_in, &L.m_in));
-			XALM_TRY(upload_vec(m, p + "mix.dq.norm", &L.dq_norm));
-			XALM_TRY(upload_rows(m, {T(p + "mix.uq")}, Rq, false, &L.w_uq, &L.m_uq));
-			XALM_TRY(upload_transposed_heads(m, T(p + "mix.uk"), H, d, R, &L.w_ukT));
-			XALM_TRY(upload_rows(m, {T(p + "mix.uv")}, R, false, &L.w_uv, nullptr));
-			if (own) {
-				XALM_TRY(upload_vec(m, p + "mix.dkv.norm", &L.dkv_norm));
-				L.cache_ld = R + r;
-				uint8_t* cache = nullptr;
-				XALM_TRY(dev_alloc(m, &cache, (size_t) m->max_tokens * L.cache_ld * kelem, true));
-				L.cache = cache;
-			} else {
-				L.cache = m->layers[(size_t) L.kv_from].cache;
-				L.cache_ld = m->layers[(size_t) L.kv_from].cache_ld;
-			}
-			// the attention sees one key/value head of R + r (values: R)
-			if (!swa_pick_tq(H, 1, R + r, R, m->chunk) && swa_smem_bytes(H, R + r, R) > 200 * 1024)
-				return set_error(XALM_ERR_UNSUPPORTED, "layer %zu: %d heads over a latent of %d + %d need %zu bytes of shared memory", li, H, R, r, swa_smem_bytes(H, R + r, R));
-			XALM_TRY(swa_prepare(H, R + r, R));
-			max_cq = std::max(max_cq, (size_t) Rq);
-			max_q = std::max(max_q, (size_t) H * (d + r));
-			max_qabs = std::max(max_qabs, (size_t) H * (R + r));
-			max_olat = std::max(max_olat, (size_t) H * R);
-			max_h = std::max(max_h, (size_t) H);
+			XALM_TRY(latent_upload(m, p + "mix.", li, &L.lat, &m->lat, &m->parts));
+			if (L.kv_from < 0) XALM_TRY(latent_cache_alloc(m, L.lat, &L.cache));
+			else L.cache = m->layers[(size_t) L.kv_from].cache;
+			max_in = std::max(max_in, (size_t) L.lat.n_in);
 		}
 		XALM_TRY(upload_rows(m, {T(p + "mix.o")}, H * dv, false, &L.w_o, &L.m_o));
 		max_in = std::max(max_in, (size_t) L.n_in);
@@ -428,9 +329,9 @@ int finalize(SeqModel* sm) {
 	}
 	XALM_TRY(hc_norm_prepare(W));
 	for (Layer& L : m->layers) {
-		XALM_TRY(tc_register(m, L.m_in, &L.t_in));
+		if (L.mixer == MIX_RETENTION) XALM_TRY(tc_register(m, L.m_in, &L.t_in));
+		else XALM_TRY(latent_tc_register(m, &L.lat));
 		XALM_TRY(tc_register(m, L.m_o, &L.t_o));
-		if (L.mixer != MIX_RETENTION) XALM_TRY(tc_register(m, L.m_uq, &L.t_uq));
 		if (L.ff_kind == FF_DENSE) {
 			XALM_TRY(tc_register(m, L.m_up, &L.t_up));
 			XALM_TRY(tc_register(m, L.m_down, &L.t_down));
@@ -438,19 +339,13 @@ int finalize(SeqModel* sm) {
 		if (L.ff_kind == FF_MOE) XALM_TRY(moe_tc_register(m, &L.moe, &m->moe));
 	}
 	m->proj_ld = (int) ((max_in + 3) / 4 * 4);
-	m->part_cap = std::max(4 * 64, 4 * m->chunk); // one-token steps: up to 64 key splits; passes of a prompt: up to 4 per token
 	XALM_TRY(dev_alloc(m, &m->x, C * W));
 	XALM_TRY(dev_alloc(m, &m->hn, C * W));
 	XALM_TRY(dev_alloc(m, &m->proj, C * m->proj_ld));
-	XALM_TRY(dev_alloc(m, &m->cq, C * max_cq));
-	XALM_TRY(dev_alloc(m, &m->q, C * max_q));
-	XALM_TRY(dev_alloc(m, &m->qabs, C * max_qabs));
-	XALM_TRY(dev_alloc(m, &m->olat, C * max_olat));
+	XALM_TRY(latent_alloc(m, &m->lat));
 	XALM_TRY(dev_alloc(m, &m->att, C * max_att));
 	XALM_TRY(dev_alloc(m, &m->ffh, C * max_ff));
-	XALM_TRY(dev_alloc(m, &m->part_o, (size_t) m->part_cap * max_olat));
-	XALM_TRY(dev_alloc(m, &m->part_ml, (size_t) m->part_cap * 2 * max_h));
-	XALM_TRY(dev_alloc(m, &m->tickets, 8 * C, true)); // the heads of a layer may run in up to 8 launches, each with counters of its own
+	XALM_TRY(attn_parts_alloc(m, &m->parts));
 	return moe_alloc(m, &m->moe);
 }
 
@@ -468,7 +363,7 @@ long long active_bytes(SeqModel* sm, long long pos) {
 	const long long kelem = m->precision == XALM_PRECISION_F32 ? 4 : 2, welem = m->w_bf16 ? 2 : 4;
 	for (const Layer& L : m->layers) {
 		if (L.mixer == MIX_RETENTION) b += 2ll * L.H * L.d * L.dv * 4;
-		else b += (pos + 1) * (L.R + L.r) * kelem;
+		else b += (pos + 1) * (L.lat.R + L.lat.r) * kelem;
 		if (L.ff_kind == FF_MOE) b -= (long long) (L.moe.E - L.moe.top) * 3 * L.moe.ff * m->width * welem;
 	}
 	return b;
@@ -486,7 +381,8 @@ bool state_buffer(SeqModel* sm, int layer, const float** src, size_t* count) {
 void destroy(SeqModel* sm) {
 	Du* m = static_cast<Du*>(sm);
 	for (Layer& L : m->layers) {
-		for (TcWeight* t : {&L.t_in, &L.t_o, &L.t_uq, &L.t_up, &L.t_down}) tc_weight_free(t);
+		for (TcWeight* t : {&L.t_in, &L.t_o, &L.t_up, &L.t_down}) tc_weight_free(t);
+		latent_free(&L.lat);
 		moe_free(&L.moe);
 	}
 	delete m;

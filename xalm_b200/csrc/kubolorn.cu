@@ -247,17 +247,12 @@ int parse_config(SeqModel* sm, const char* json) {
 			m->layers.push_back(std::move(L));
 		}
 		// the order the layers run in: layers start .. stop - 1 `times` times in a row, then the rest
-		const int nl = (int) m->layers.size();
-		int start = 0, stop = 0, times = 1;
-		if (const xjson::Value* lp = c.find("loop"); lp && lp->kind == xjson::Value::Obj) {
-			start = geti(*lp, "start"); stop = geti(*lp, "stop"); times = lp->contains("times") ? geti(*lp, "times") : 1;
-			if (start < 0 || stop < start || stop > nl || times < 1) return set_error(XALM_ERR_INVALID, "config: loop over layers [%d, %d) %d times", start, stop, times);
-		}
-		for (int li = 0; li < nl; li++) {
-			if (li == start && stop > start)
-				for (int r = 0; r < times; r++)
-					for (int lj = start; lj < stop; lj++) { Run R; R.layer = lj; m->runs.push_back(R); }
-			if (li < start || li >= stop) { Run R; R.layer = li; m->runs.push_back(R); }
+		std::vector<LayerRun> order;
+		XALM_TRY(layer_order(c, (int) m->layers.size(), &order));
+		for (const LayerRun& r : order) {
+			Run R;
+			R.layer = r.layer;
+			m->runs.push_back(R);
 		}
 		m->n_layers = (int) m->runs.size(); // what read_state counts: layer runs
 		expect(m, "final.norm", {W}, false);

@@ -17,6 +17,7 @@
 //   dual_norm_hc_kernel    y = 1/2 (rmsnorm(a) wa + rmsnorm(b) wb) -> layer scale -> hyper-connection write
 //   group_norm_residual_kernel  x + grouped RMS norm of a sublayer's output (weighted sum of expert rows first), depth-weighted average
 //   qkv_post_kernel        bias, rotary positions, RMS norms of q / k / v heads, query temperature, K/V cache write (kept first slots + ring)
+//   qkv_rows_post_kernel   RMS norms of the whole q and k rows (all heads together), then rotary positions, K/V cache write
 //   layer_norm_kernel      (x - mean) / sqrt(variance + eps) * w + b
 //
 // The kernels have internal linkage: every translation unit that includes this header (a model family, the op-level entry points
@@ -516,6 +517,8 @@ struct SwaArgs {
 	int window;        // position i sees j with 0 <= i - j < window
 	int keep_first;    // ... and every j < keep_first (j <= i) however far back: the sequence's first positions stay visible at their true
 	                   // places.  They live in slots [0, keep_first) of the cache, the others in the `ring` slots behind (0: a plain ring)
+	int mask_chunk;    // > 0: the sequence is cut into runs of mask_chunk positions from position 0 on, and a query sees its own run only (up to
+	                   // itself; the window still applies).  Not together with keep_first.  0: one run
 	float scale;
 	float softcap;     // 0: none
 	const float* r1;   // distance bias r1[h] * log1p(r2[h] * (i - j)) taken off the score; NULL: none
@@ -551,9 +554,11 @@ struct SwaKeys {
 		return j < keep ? j : keep + (j - keep) % ring;
 	}
 };
-__device__ __forceinline__ SwaKeys swa_keys(int window, int keep_first, int ring, int i_lo) {
+__device__ __forceinline__ SwaKeys swa_keys(const SwaArgs& a, int i_lo) {
+	const int keep_first = a.keep_first, ring = a.ring;
 	SwaKeys k;
-	k.j_first = window < 0x7fffffff ? max(0, i_lo - window + 1) : 0;
+	k.j_first = a.window < 0x7fffffff ? max(0, i_lo - a.window + 1) : 0;
+	if (a.mask_chunk > 0) k.j_first = max(k.j_first, i_lo - i_lo % a.mask_chunk);
 	k.ks = min(keep_first, k.j_first);
 	k.keep = keep_first;
 	k.ring = ring;
@@ -662,7 +667,7 @@ __global__ void __launch_bounds__(256) swa_attn_kernel(SwaArgs a) {
 	const bool vec8 = ((d | ldk) & 7) == 0 && (reinterpret_cast<uintptr_t>(a.kc) & 31) == 0;
 	if (t >= a.step->n) return;
 	const int i = a.step->pos0 + t;
-	const SwaKeys km = swa_keys(a.window, a.keep_first, a.ring, i);
+	const SwaKeys km = swa_keys(a, i);
 	const int nk = km.ks + i - km.j_first + 1; // every one of them is visible to this query
 	int per = (nk + a.n_splits - 1) / a.n_splits;
 	per = (per + SWA_KB - 1) / SWA_KB * SWA_KB;
@@ -1021,7 +1026,7 @@ __global__ void __launch_bounds__(256) swa_tile_kernel(SwaArgs a) {
 	const int nq = min(TQ, n - t0);          // queries of this tile (<= 0: nothing to do)
 	if (nq <= 0) return;
 	const int i_lo = pos0 + t0, i_hi = i_lo + nq - 1;
-	const SwaKeys km = swa_keys(a.window, a.keep_first, a.ring, i_lo);
+	const SwaKeys km = swa_keys(a, i_lo);
 	const int nk = km.ks + i_hi - km.j_first + 1;
 	int per = (nk + a.n_splits - 1) / a.n_splits;
 	per = (per + SWA_KB - 1) / SWA_KB * SWA_KB;
@@ -1079,7 +1084,8 @@ __global__ void __launch_bounds__(256) swa_tile_kernel(SwaArgs a) {
 				m4[0] = fmaf(w.x, s, m4[0]); m4[1] = fmaf(w.y, s, m4[1]); m4[2] = fmaf(w.z, s, m4[2]); m4[3] = fmaf(w.w, s, m4[3]);
 			}
 			const int i = i_lo + q, j = km.pos(j0 + jj);
-			const bool seen = q < nq && jj < nbk && j <= i && (a.window >= 0x7fffffff || i - j < a.window || j < a.keep_first);
+			const bool seen = q < nq && jj < nbk && j <= i && (a.window >= 0x7fffffff || i - j < a.window || j < a.keep_first) &&
+			                  (a.mask_chunk <= 0 || j >= i - i % a.mask_chunk);
 #pragma unroll
 			for (int u = 0; u < 4; u++) {
 				const int h = 4 * hq + u;
@@ -1737,6 +1743,8 @@ static inline int launch_group_norm(const GroupNormArgs& a, int rows, cudaStream
 // dimensions of a query / key head, dimension i paired with i + rot_half, angle = position * freq[i] in fp32 (sincosf).  The norms
 // (x / sqrt(mean(x^2) + eps) over the head; q_norm_w / k_norm_w: a weight over the head's entries, shared by all heads) come after the
 // rotation; each is optional.  Last, a query at position p is multiplied by 1 + temp_coef * ln(floor((p + 1) / temp_every) + 1) when temp_every > 0.
+// With norm_rows the norms are over the whole q and the whole k row, with a weight per entry, and come BEFORE the rotation: a kernel of its own
+// (qkv_rows_post_kernel below), which also turns neighbouring entries (2i, 2i + 1) as a pair when rot_neighbours is set.
 struct QkvPostArgs {
 	float* proj; // (T, ld)
 	int ld, q_off, k_off, v_off;
@@ -1746,7 +1754,10 @@ struct QkvPostArgs {
 	int rot_half;
 	float rot_mag;             // multiplies cos and sin of every turn (a rescaled rotation changes the length of what it turns); 0: 1
 	int norm_qk, norm_v;
-	const float *q_norm_w, *k_norm_w; // (d) or NULL (weight 1)
+	const float *q_norm_w, *k_norm_w; // (d) or NULL (weight 1); norm_rows: (H * d) and (G * d)
+	int norm_rows, rot_neighbours;
+	float* q_out; // norm_rows: (T, ldq_out) the finished queries, or NULL: in place
+	int ldq_out;
 	int temp_every;
 	float temp_coef;
 	float eps;
@@ -1807,7 +1818,89 @@ static __global__ void qkv_post_kernel(QkvPostArgs a) {
 	else
 		for (int c = lane; c < n; c += 32) ((__nv_bfloat16*) cache)[at + c] = __float2bfloat16_rn(x[c] * rs);
 }
+// grid (rows, parts), 256 threads; shared memory: 2 * rot_half + 33 floats.  Every CTA sums the squares of whole rows (of the rows its share needs) and
+// finishes its share of the (entry, entry) pairs, so that a one-token step spreads over several CTAs; that needs q_out apart from proj.
+static __global__ void qkv_rows_post_kernel(QkvPostArgs a) {
+	extern __shared__ float sm[];
+	float *cs = sm, *sn = sm + a.rot_half, *red = sn + a.rot_half;
+	const int t = blockIdx.x, tid = threadIdx.x, nth = blockDim.x;
+	if (t >= a.step->n) return;
+	const int pos = a.step->pos0 + t, r = a.freq ? a.rot_half : 0;
+	float* row = a.proj + (size_t) t * a.ld;
+	float* q_out = a.q_out ? a.q_out + (size_t) t * a.ldq_out : row + a.q_off;
+	for (int c = tid; c < r; c += nth) sincosf((float) pos * a.freq[c], &sn[c], &cs[c]);
+	// units: pairs of query entries, pairs of key entries, value entries
+	const int dp = (a.d + 1) / 2, nq = a.H * dp, nk = a.G * dp, units = nq + nk + a.G * a.dv;
+	const int per = (units + (int) gridDim.y - 1) / (int) gridDim.y, u0 = blockIdx.y * per, u1 = min(units, u0 + per);
+	float inv[2] = {1.f, 1.f};
+	if (a.norm_rows)
+		for (int k = 0; k < 2; k++) { // uniform over the CTA
+			if (k ? !(u1 > nq && u0 < nq + nk) : u0 >= nq) continue;
+			const float* src = row + (k ? a.k_off : a.q_off);
+			const int n = (k ? a.G : a.H) * a.d;
+			float ss = 0.f;
+			if (((n | (k ? a.k_off : a.q_off) | a.ld) & 3) == 0) {
+#pragma unroll 4
+				for (int c = tid * 4; c < n; c += nth * 4) {
+					const float4 v = *reinterpret_cast<const float4*>(src + c);
+					ss = fmaf(v.x, v.x, ss); ss = fmaf(v.y, v.y, ss); ss = fmaf(v.z, v.z, ss); ss = fmaf(v.w, v.w, ss);
+				}
+			} else
+				for (int c = tid; c < n; c += nth) ss = fmaf(src[c], src[c], ss);
+			inv[k] = 1.f / sqrtf(block_sum(ss, red) / (float) n + a.eps);
+		}
+	__syncthreads(); // the table of turns is complete, and every sum has read the rows that may now be overwritten
+	const int slot = pos < a.keep_first ? pos : a.keep_first + (pos - a.keep_first) % a.ring;
+	for (int u = u0 + tid; u < u1; u += nth) {
+		if (u >= nq + nk) {
+			const int c = u - nq - nk;
+			const size_t at = (size_t) slot * a.G * a.dv + c;
+			const float v = row[a.v_off + c];
+			if (a.cache_f32) ((float*) a.vc)[at] = v;
+			else ((__nv_bfloat16*) a.vc)[at] = __float2bfloat16_rn(v);
+			continue;
+		}
+		const bool is_k = u >= nq;
+		const int x = is_k ? u - nq : u, hd = x / dp, p = x % dp;
+		// pairs behind the rotated ones are neighbours in either layout (2 rot_half entries lie before them)
+		const int i0 = a.rot_neighbours || p >= r ? 2 * p : p, i1 = a.rot_neighbours || p >= r ? 2 * p + 1 : p + r;
+		const int e0 = hd * a.d + i0, e1 = hd * a.d + i1;
+		const bool two = i1 < a.d;
+		const float* src = row + (is_k ? a.k_off : a.q_off);
+		const float* w = is_k ? a.k_norm_w : a.q_norm_w;
+		const float rs = is_k ? inv[1] : inv[0];
+		float v0 = src[e0] * rs, v1 = two ? src[e1] * rs : 0.f;
+		if (w) { v0 *= w[e0]; v1 *= two ? w[e1] : 0.f; }
+		if (p < r) {
+			const float c = cs[p], s = sn[p], y0 = v0 * c - v1 * s;
+			v1 = v1 * c + v0 * s;
+			v0 = y0;
+		}
+		if (!is_k) {
+			q_out[e0] = v0;
+			if (two) q_out[e1] = v1;
+		} else {
+			const size_t at = (size_t) slot * a.G * a.d;
+			if (a.cache_f32) {
+				((float*) a.kc)[at + e0] = v0;
+				if (two) ((float*) a.kc)[at + e1] = v1;
+			} else {
+				((__nv_bfloat16*) a.kc)[at + e0] = __float2bfloat16_rn(v0);
+				if (two) ((__nv_bfloat16*) a.kc)[at + e1] = __float2bfloat16_rn(v1);
+			}
+		}
+	}
+}
 static inline int launch_qkv_post(const QkvPostArgs& a, int rows, cudaStream_t s) {
+	if (a.norm_rows || a.rot_neighbours) {
+		if (a.bq || a.bk || a.bv || a.norm_qk || a.norm_v || a.temp_every > 0 || a.rot_mag != 0.f)
+			return set_error(XALM_ERR_UNSUPPORTED, "qkv_post: row norms or neighbouring pairs together with biases, head norms, temperature or rotation magnitude");
+		if (a.rot_half < 0 || 2 * a.rot_half > a.d || (size_t) a.rot_half * 8 > 40 * 1024) return set_error(XALM_ERR_INVALID, "qkv_post: %d pairs in a head of %d", a.rot_half, a.d);
+		const int units = (a.H + a.G) * ((a.d + 1) / 2) + a.G * a.dv;
+		const int parts = a.q_out && rows < 64 ? std::max(1, std::min(8, units / 512)) : 1; // short steps: several CTAs per token
+		qkv_rows_post_kernel<<<dim3(rows, parts), 256, ((size_t) 2 * a.rot_half + 33) * 4, s>>>(a);
+		return launch_check("qkv_rows_post");
+	}
 	const int units = a.H + 2 * a.G, nw = units < 8 ? units : 8, wmax = a.d > a.dv ? a.d : a.dv;
 	if ((size_t) nw * wmax * 4 > 48 * 1024) return set_error(XALM_ERR_UNSUPPORTED, "qkv_post: heads of %d do not fit shared memory", wmax);
 	qkv_post_kernel<<<dim3(rows, (units + nw - 1) / nw), nw * 32, (size_t) nw * wmax * 4, s>>>(a);
@@ -1884,6 +1977,7 @@ static inline int swa_pick_tq(int H, int G, int d, int dv, int rows) {
 // rows: tokens of the step; cache_f32: element type of the ring.  With n_splits > 1 the merge kernel follows.  Returns the number of
 // launches through *launches (1 or 2) when it is given.
 static inline int launch_swa(SwaArgs a, int rows, bool cache_f32, cudaStream_t s, int* launches = nullptr) {
+	if (a.mask_chunk > 0 && a.keep_first > 0) return set_error(XALM_ERR_UNSUPPORTED, "attention: kept first positions together with chunks");
 	// One key/value group, no score mixing, more than a few rows, and all heads together do not fit a CTA's shared memory in the tiled kernel
 	// (many heads over a wide latent): the heads run in 2, 4 or 8 launches, each a smaller attention of its own on its share of the query
 	// and output columns, with its own slice of the partial buffers and ticket counters.
@@ -1916,7 +2010,9 @@ static inline int launch_swa(SwaArgs a, int rows, bool cache_f32, cudaStream_t s
 	const int tq = swa_pick_tq(a.H, a.G, a.d, a.dv, rows);
 	if (a.n_splits <= 0) { // enough CTAs for two waves, at least two key blocks each
 		const int qblocks = tq ? (rows + tq - 1) / tq : rows;
-		const long long keys = std::min<long long>((long long) a.ring, (long long) (a.window < 0x7fffffff ? a.window : a.ring) + (tq ? tq : 1)) + a.keep_first;
+		long long reach = a.window < 0x7fffffff ? a.window : a.ring;
+		if (a.mask_chunk > 0) reach = std::min<long long>(reach, a.mask_chunk);
+		const long long keys = std::min<long long>((long long) a.ring, reach + (tq ? tq : 1)) + a.keep_first;
 		int want = std::max(1, 296 / std::max(1, qblocks));
 		want = (int) std::min<long long>(want, std::max<long long>(1, tq ? keys / (2 * SWA_KB) : (keys + SWA_KB - 1) / SWA_KB)); // key blocks per CTA: >= 2 (tiled), 1 (one query)
 		a.n_splits = (a.part_o && a.part_ml) ? std::max(1, std::min(want, a.part_cap / std::max(1, rows))) : 1;

@@ -49,10 +49,6 @@ struct Layer { // weights and sizes; what a sequence holds lives in Run
 	TcWeight t_in, t_o;
 	bool has_moe = false;
 	MoeWeights moe;
-	int shared_ff = 0; // 0: no shared expert
-	void *w_sup = nullptr, *w_sdown = nullptr;
-	WMat m_sup, m_sdown;
-	TcWeight t_sup, t_sdown;
 	long long bytes = 0, expert_bytes = 0; // what one run of the layer reads of its matrices; of that, one expert's share
 };
 
@@ -73,7 +69,7 @@ struct MizeraxModel : SeqModel {
 	TcWeight t_lx, t_l0;
 	float* final_norm_b = nullptr;
 	// one pass
-	float *x = nullptr, *x2 = nullptr, *x0w = nullptr, *hn = nullptr, *proj = nullptr, *att = nullptr, *ao = nullptr, *shid = nullptr, *sout = nullptr;
+	float *x = nullptr, *x2 = nullptr, *x0w = nullptr, *hn = nullptr, *proj = nullptr, *att = nullptr, *ao = nullptr;
 	int proj_ld = 4;
 	float *part_o = nullptr, *part_ml = nullptr;
 	unsigned* tickets = nullptr;
@@ -83,11 +79,6 @@ struct MizeraxModel : SeqModel {
 typedef MizeraxModel Mz;
 
 // ---- config.json ------------------------------------------------------------------------------------------------------------------
-const xjson::Value* object_or_null(const xjson::Value& o, const char* k) {
-	const xjson::Value* v = o.find(k);
-	return v && v->kind == xjson::Value::Obj ? v : nullptr;
-}
-
 int parse_layer(Mz* m, size_t li, const xjson::Value& lv) {
 	const int W = m->width;
 	const std::string p = "l" + std::to_string(li) + ".", type = lv.at("type").str;
@@ -132,11 +123,9 @@ int parse_layer(Mz* m, size_t li, const xjson::Value& lv) {
 		expect(m, p + "mlp.router", {e.E + e.identity, W}, true);
 		expect(m, p + "mlp.correction", {e.E + e.identity}, false);
 		if (const xjson::Value* sh = object_or_null(*mlp, "shared")) {
-			L.shared_ff = geti(*sh, "ff");
-			if (L.shared_ff <= 0) return set_error(XALM_ERR_INVALID, "config: layer %zu: shared expert of %d", li, L.shared_ff);
-			expect(m, p + "mlp.shared.gate", {L.shared_ff, W}, true);
-			expect(m, p + "mlp.shared.up", {L.shared_ff, W}, true);
-			expect(m, p + "mlp.shared.down", {W, L.shared_ff}, true);
+			const int sff = geti(*sh, "ff");
+			if (sff <= 0) return set_error(XALM_ERR_INVALID, "config: layer %zu: shared expert of %d", li, sff);
+			moe_expect_shared(m, p + "mlp.shared.", &e, sff, false);
 		}
 		expect(m, p + "ls2", {W}, false);
 	}
@@ -160,25 +149,16 @@ int parse_config(SeqModel* sm, const char* json) {
 		const xjson::Value& layers = c.at("layers");
 		if (layers.kind != xjson::Value::Array || layers.arr.empty()) return set_error(XALM_ERR_INVALID, "config: no layers");
 		for (size_t li = 0; li < layers.arr.size(); li++) XALM_TRY(parse_layer(m, li, layers.arr[li]));
-		// the order the layers run in: layers start .. stop - 1 `times` times in a row, then the rest
-		const int nl = (int) m->layers.size();
-		int start = 0, stop = 0, times = 1;
-		if (const xjson::Value* lp = object_or_null(c, "loop")) {
-			start = geti(*lp, "start"); stop = geti(*lp, "stop"); times = lp->contains("times") ? geti(*lp, "times") : 1;
-			if (start < 0 || stop < start || stop > nl || times < 1) return set_error(XALM_ERR_INVALID, "config: loop over layers [%d, %d) %d times", start, stop, times);
-			m->loops = stop > start;
-			if (m->loops) expect(m, "loop.in", {m->width, 2 * m->width}, true);
-		}
-		auto add_run = [&](int layer, bool begins) {
+		std::vector<LayerRun> order;
+		XALM_TRY(layer_order(c, (int) m->layers.size(), &order));
+		for (const LayerRun& r : order) {
 			Run R;
-			R.layer = layer;
-			R.begins = begins;
+			R.layer = r.layer;
+			R.begins = r.pass > 0; // every pass over the loop begins with loop.in's product
+			m->loops = m->loops || R.begins;
 			m->runs.push_back(R);
-		};
-		for (int li = 0; li < start; li++) add_run(li, false);
-		for (int r = 0; r < times; r++)
-			for (int li = start; li < stop; li++) add_run(li, li == start);
-		for (int li = stop; li < nl; li++) add_run(li, false);
+		}
+		if (m->loops) expect(m, "loop.in", {m->width, 2 * m->width}, true);
 		m->n_layers = (int) m->runs.size(); // what read_state counts: layer runs
 		expect(m, "final.norm", {m->width}, false);
 		expect(m, "final.norm.b", {m->width}, false);
@@ -220,20 +200,11 @@ int enqueue_attention(Mz* m, const Layer& L, const Run& R, int n, const Fork& fk
 
 // experts and shared expert of m->hn; *ca names everything the join adds
 int enqueue_mixture(Mz* m, const Layer& L, int n, MoeCombineArgs* ca, int* nl) {
-	const int W = m->width;
 	MoeRouteArgs ra = {};
 	ra.score_kind = MOE_SCORE_SOFTMAX; // the weights are the scores themselves
 	RowsEpi eg;
 	eg.kind = EPI_GLU; eg.glu_act = GLU_SILU;
 	XALM_TRY(moe_experts(m, L.moe, m->moe, m->hn, n, ra, eg, ca, nl));
-	if (L.shared_ff) {
-		eg.out = m->shid; eg.ldo = L.shared_ff;
-		XALM_TRY(rows_product(m, m->hn, W, L.w_sup, &L.t_sup, n, 2 * L.shared_ff, W, eg, nl));
-		RowsEpi es;
-		es.kind = EPI_STORE; es.out = m->sout; es.ldo = W;
-		XALM_TRY(rows_product(m, m->shid, L.shared_ff, L.w_sdown, &L.t_sdown, n, W, L.shared_ff, es, nl));
-		ca->base = m->sout;
-	}
 	ca->scale = L.ls2;
 	return XALM_OK;
 }
@@ -315,7 +286,7 @@ int finalize(SeqModel* sm) {
 	const int W = m->width;
 	const size_t C = (size_t) m->chunk, kelem = m->precision == XALM_PRECISION_F32 ? 4 : 2;
 	auto T = [&](const std::string& n) { return tensor_or_null(m, n); };
-	size_t max_in = 4, max_att = 1, max_h = 1, max_shared = 1;
+	size_t max_in = 4, max_att = 1, max_h = 1;
 	XALM_TRY(upload_rows(m, {T("pos")}, W, false, &m->positions, nullptr));
 	XALM_TRY(upload_vec(m, "final.norm.b", &m->final_norm_b));
 	if (m->loops) { // loop.in's columns: the left half reads x, the right half the embedded row
@@ -358,11 +329,6 @@ int finalize(SeqModel* sm) {
 			XALM_TRY(upload_vec(m, p + "mlp.correction", &L.moe.correction));
 			XALM_TRY(moe_upload(m, p + "mlp.", true, &L.moe, &m->moe));
 			L.expert_bytes = 3ll * L.moe.ff * W * (m->w_bf16 ? 2 : 4);
-			if (L.shared_ff) {
-				XALM_TRY(upload_rows(m, {T(p + "mlp.shared.gate"), T(p + "mlp.shared.up")}, W, true, &L.w_sup, &L.m_sup));
-				XALM_TRY(upload_rows(m, {T(p + "mlp.shared.down")}, L.shared_ff, false, &L.w_sdown, &L.m_sdown));
-				max_shared = std::max(max_shared, (size_t) L.shared_ff);
-			}
 		}
 		L.bytes = m->weight_bytes - bytes0;
 		max_in = std::max(max_in, (size_t) L.n_in);
@@ -378,10 +344,6 @@ int finalize(SeqModel* sm) {
 		XALM_TRY(tc_register(m, L.m_in, &L.t_in));
 		XALM_TRY(tc_register(m, L.m_o, &L.t_o));
 		if (L.has_moe) XALM_TRY(moe_tc_register(m, &L.moe, &m->moe));
-		if (L.shared_ff) {
-			XALM_TRY(tc_register(m, L.m_sup, &L.t_sup));
-			XALM_TRY(tc_register(m, L.m_sdown, &L.t_sdown));
-		}
 	}
 	// what the sequence holds, per layer run
 	for (Run& R : m->runs) {
@@ -400,8 +362,6 @@ int finalize(SeqModel* sm) {
 	XALM_TRY(dev_alloc(m, &m->proj, C * m->proj_ld));
 	XALM_TRY(dev_alloc(m, &m->att, C * max_att));
 	XALM_TRY(dev_alloc(m, &m->ao, C * W));
-	XALM_TRY(dev_alloc(m, &m->shid, C * max_shared));
-	XALM_TRY(dev_alloc(m, &m->sout, C * W));
 	XALM_TRY(dev_alloc(m, &m->part_o, (size_t) m->part_cap * max_att));
 	XALM_TRY(dev_alloc(m, &m->part_ml, (size_t) m->part_cap * 2 * max_h));
 	XALM_TRY(dev_alloc(m, &m->tickets, 8 * C, true));
@@ -437,7 +397,7 @@ void destroy(SeqModel* sm) {
 	tc_weight_free(&m->t_lx);
 	tc_weight_free(&m->t_l0);
 	for (Layer& L : m->layers) {
-		for (TcWeight* t : {&L.t_in, &L.t_o, &L.t_sup, &L.t_sdown}) tc_weight_free(t);
+		for (TcWeight* t : {&L.t_in, &L.t_o}) tc_weight_free(t);
 		moe_free(&L.moe);
 	}
 	delete m;

@@ -4,9 +4,10 @@
 //                       experts form n_groups equal groups of neighbours, a group scores the sum of its two largest s or its largest s, and
 //                       only experts of the keep_groups best groups can be chosen; the `top` largest s among those are chosen (ties: the
 //                       lower index); their weights are the scores themselves, or the scores over their sum.  An optional correction per
-//                       expert is added to the score for the choice alone
+//                       expert is added to the score for the choice alone.  Or the scores are the logits themselves (with an optional bias) and the
+//                       weights the softmax over the chosen ones.  A further row behind the experts' can give a gate per token, sigmoid(w h)
 //   moe_combine_kernel  x <- x + sum of a token's `top` expert rows with their weights, in slot order (identity experts contribute the mixture's
-//                       input row), optionally with a shared expert's row, a second sublayer's row and a scale per column
+//                       input row), optionally with a shared expert's row (times a gate per token), a second sublayer's row and a scale per column
 //   moe_sort_kernel     the step's (token, slot) pairs ordered by expert, cut into row tiles of one expert each; the pairs of experts without
 //                       matrices (identity experts, numbered behind the others) come last and get no tile
 //   moe_gemm_kernel     out[pair] = A[row of pair] . W_expert(pair)^T in IEEE fp32 for every tile, with the row products' fused epilogues
@@ -34,13 +35,16 @@ struct MoeRouteArgs {
 	int* idx;   // (T, top)
 	float* wgt; // (T, top)
 	const SeqStep* step;
-	int score_kind;  // MOE_SCORE_SIGMOID (0) or MOE_SCORE_SOFTMAX: exp(z - max z) / sum over all experts
+	int score_kind;  // MOE_SCORE_SIGMOID (0), MOE_SCORE_SOFTMAX: exp(z - max z) / sum over all experts, or MOE_SCORE_CHOSEN: z itself is compared, and the
+	                 // weights are exp(z - max z) / sum over the chosen experts
 	int group_kind;  // MOE_GROUP_TOP2_SUM (0) or MOE_GROUP_MAX: what a group scores
 	int renormalise; // 1: the chosen weights are divided by (their sum + renorm_eps)
 	float renorm_eps;
 	const float* correction; // (E) added to the scores where they are compared, not where they become weights; NULL: none.  Without groups
+	const float* bias;       // (E) added to the logits; NULL: none
+	float* gate_out;         // (T) sigmoid of row E of w times h: a gate of a shared expert, computed where h is at hand; NULL: w has no such row
 };
-enum { MOE_SCORE_SIGMOID = 0, MOE_SCORE_SOFTMAX = 1 };
+enum { MOE_SCORE_SIGMOID = 0, MOE_SCORE_SOFTMAX = 1, MOE_SCORE_CHOSEN = 2 };
 enum { MOE_GROUP_TOP2_SUM = 0, MOE_GROUP_MAX = 1 };
 
 // (value, index) argmax over a warp; ties go to the lower index; index -1 = nothing
@@ -65,7 +69,7 @@ __global__ void __launch_bounds__(256) moe_router_kernel(MoeRouteArgs a) {
 	for (int k = tid; k < a.K; k += nth) hs[k] = a.h[(size_t) t * a.ldh + k];
 	__syncthreads();
 	const WT* W = reinterpret_cast<const WT*>(a.w);
-	for (int e = warp; e < a.E; e += nw) {
+	for (int e = warp; e < a.E + (a.gate_out ? 1 : 0); e += nw) {
 		float z = 0.f;
 		if ((a.K & 7) == 0 && (reinterpret_cast<uintptr_t>(a.w) & 31) == 0) {
 #pragma unroll 4
@@ -78,7 +82,13 @@ __global__ void __launch_bounds__(256) moe_router_kernel(MoeRouteArgs a) {
 		} else
 			for (int k = lane; k < a.K; k += 32) z = fmaf(ldf(W + (size_t) e * a.K + k), hs[k], z);
 		z = warp_sum(z);
-		if (lane == 0) sc[e] = a.score_kind == MOE_SCORE_SOFTMAX ? z : sigmoidf_(z);
+		if (lane == 0) {
+			if (e == a.E) a.gate_out[t] = sigmoidf_(z);
+			else {
+				if (a.bias) z += a.bias[e];
+				sc[e] = a.score_kind == MOE_SCORE_SIGMOID ? sigmoidf_(z) : z;
+			}
+		}
 	}
 	__syncthreads();
 	if (warp != 0) return;
@@ -135,6 +145,15 @@ __global__ void __launch_bounds__(256) moe_router_kernel(MoeRouteArgs a) {
 		}
 		__syncwarp();
 	}
+	if (a.score_kind == MOE_SCORE_CHOSEN) { // the first choice has the largest logit
+		const size_t at = (size_t) t * a.top;
+		const float zm = a.wgt[at];
+		__syncwarp();
+		float tot = 0.f;
+		for (int r = lane; r < a.top; r += 32) tot += expf(a.wgt[at + r] - zm);
+		tot = warp_sum(tot);
+		for (int r = lane; r < a.top; r += 32) a.wgt[at + r] = expf(a.wgt[at + r] - zm) / tot;
+	}
 	if (a.renormalise) {
 		float tot = 0.f;
 		for (int r = lane; r < a.top; r += 32) tot += a.wgt[(size_t) t * a.top + r]; // written by lane 0 above
@@ -157,6 +176,7 @@ struct MoeCombineArgs {
 	int n_experts;
 	const float* ident;  // (rows, width)
 	const float* base;   // (rows, width) added to the weighted sum (a shared expert's output), or NULL
+	const float* base_w; // (rows) multiplies base's row, or NULL
 	const float* scale;  // (width) multiplies the sum, or NULL
 	const float* other;  // (rows, width) a sublayer beside the mixture: other_scale[c] * other[t][c] is added as well, or NULL
 	const float* other_scale;
@@ -173,7 +193,7 @@ static __global__ void moe_combine_kernel(MoeCombineArgs a) {
 			const float y = a.idx && a.idx[pk] >= a.n_experts ? a.ident[at] : a.y[(a.part_row ? (size_t) a.part_row[pk] : pk) * a.ldy + c];
 			v = fmaf(a.wgt[pk], y, v);
 		}
-		if (a.base) v += a.base[at];
+		if (a.base) v = fmaf(a.base_w ? a.base_w[t] : 1.f, a.base[at], v);
 		if (a.scale) v *= a.scale[c];
 		if (a.other) v = fmaf(a.other_scale ? a.other_scale[c] : 1.f, a.other[at], v);
 		a.x_out[at] = a.x_in ? a.x_in[at] + v : v;
@@ -379,6 +399,7 @@ static inline int launch_moe_router(const MoeRouteArgs& a, int rows, cudaStream_
 	if (a.E <= 0 || a.top <= 0 || a.top > a.E) return set_error(XALM_ERR_INVALID, "router: %d of %d experts", a.top, a.E);
 	if (a.n_groups > 1 && (a.E % a.n_groups || a.keep_groups <= 0 || a.keep_groups > a.n_groups || a.keep_groups * (a.E / a.n_groups) < a.top))
 		return set_error(XALM_ERR_INVALID, "router: %d groups, %d kept, cannot hold %d of %d experts", a.n_groups, a.keep_groups, a.top, a.E);
+	if (a.correction && a.score_kind == MOE_SCORE_CHOSEN) return set_error(XALM_ERR_UNSUPPORTED, "router: a choice correction on plain logits");
 	if (a.correction && a.n_groups > 1) return set_error(XALM_ERR_UNSUPPORTED, "router: a choice correction together with expert groups");
 	const size_t smem = moe_router_smem(a.K, a.E, a.n_groups);
 	if (a.w_bf16) moe_router_kernel<__nv_bfloat16><<<rows, 256, smem, s>>>(a);

@@ -1,5 +1,5 @@
 // seq_family.cuh — the sequence engine shared by the model families that a config.json describes (Nabalix, Bolovik, Duletar, Kubolorn,
-// Mizerax): what a family does NOT write itself.
+// Mizerax, Pavitar): what a family does NOT write itself.
 //
 //   * tensors by name: the family lists what it reads (expect), the loader uploads them (any order, fp32 / fp16 / bf16), finalize
 //     turns them into device layouts (upload_rows: several matrices stacked or interleaved into one; upload_vec);
@@ -113,6 +113,32 @@ double getf(const xjson::Value& o, const char* k) {
 	const xjson::Value& v = o.at(k);
 	if (v.kind != xjson::Value::Number) throw std::invalid_argument(std::string("config: '") + k + "' is not a number");
 	return v.num;
+}
+const xjson::Value* object_or_null(const xjson::Value& o, const char* k) {
+	const xjson::Value* v = o.find(k);
+	return v && v->kind == xjson::Value::Obj ? v : nullptr;
+}
+std::vector<float> rotary_frequencies(double base, int dims) { // f_i = base^(-2i/dims)
+	std::vector<float> f((size_t) dims / 2);
+	for (int i = 0; i < dims / 2; i++) f[(size_t) i] = (float) pow(base, -2.0 * i / dims);
+	return f;
+}
+// The order layers run in: "loop" {start, stop, times} runs layers start .. stop - 1 `times` times in a row with the same weights, then the rest.
+struct LayerRun {
+	int layer = 0;
+	int pass = 0; // the pass over the loop (from 1) that begins with this run, 0: none begins
+};
+int layer_order(const xjson::Value& c, int n_layers, std::vector<LayerRun>* out) {
+	int start = 0, stop = 0, times = 1;
+	if (const xjson::Value* lp = object_or_null(c, "loop")) {
+		start = geti(*lp, "start"); stop = geti(*lp, "stop"); times = lp->contains("times") ? geti(*lp, "times") : 1;
+		if (start < 0 || stop < start || stop > n_layers || times < 1) return set_error(XALM_ERR_INVALID, "config: loop over layers [%d, %d) %d times", start, stop, times);
+	}
+	for (int li = 0; li < start; li++) out->push_back({li, 0});
+	for (int r = 1; r <= times; r++)
+		for (int li = start; li < stop; li++) out->push_back({li, li == start ? r : 0});
+	for (int li = stop; li < n_layers; li++) out->push_back({li, 0});
+	return XALM_OK;
 }
 void expect(SeqModel* m, const std::string& name, std::vector<int> shape, bool matrix, bool required = true) {
 	HostTensor t;

@@ -3,7 +3,8 @@
 //
 //   router -> [steps of a few tokens: one matvec per (token, slot) pair] or [sort by expert -> tiled fp32 products] or, for long passes of the
 //   16-bit mode, [sort -> rows packed in expert order -> grouped tcgen05 GEMM with the activation fused -> grouped tcgen05 GEMM] on the experts'
-//   resident fp16 tiles; the caller then joins each token's expert rows (moe_combine, with whatever else its layer adds there).
+//   resident fp16 tiles; a shared expert that runs for every token (gated matrices of its own, two row products), optionally with a gate per
+//   token that the router's kernel computes; the caller then joins each token's rows (moe_combine, with whatever else its layer adds there).
 //
 // A family says what differs between designs: how scores become choices and weights (MoeRouteArgs), the activation between an expert's two
 // products (RowsEpi), how many of the router's outputs are identity experts.
@@ -22,6 +23,12 @@ struct MoeWeights {
 	int up_rows = 0;         // rows of an expert's first matrix: ff, or 2 ff when gate and up rows alternate
 	void *w_up = nullptr, *w_down = nullptr, *w_router = nullptr;
 	float* correction = nullptr; // (E + identity) or NULL
+	float* bias = nullptr;       // (E + identity) of the router's logits, or NULL
+	int shared_ff = 0;           // 0: no shared expert
+	bool shared_gate = false;    // its output is multiplied by sigmoid(w_sg h): one more row of the router's matrix
+	void *w_sup = nullptr, *w_sdown = nullptr;
+	WMat m_sup, m_sdown;
+	TcWeight t_sup, t_sdown;
 	WMat m_up, m_down;
 	std::vector<TcWeight> t_up, t_down; // per expert, when long passes run on the tensor cores
 	const uint8_t **b_up = nullptr, **b_down = nullptr; // (device) their tiles
@@ -29,11 +36,11 @@ struct MoeWeights {
 };
 
 struct MoeBuffers { // of one pass, sized for the largest mixture of the model
-	size_t max_pairs = 0, max_hid = 0;
+	size_t max_pairs = 0, max_hid = 0, max_shared = 0;
 	int max_tiles = 1;
 	size_t a_bytes = 0, h_bytes = 0; // operand planes of the tensor-core products: the mixture's input rows in expert order, the hidden rows
 	int *idx = nullptr, *sorted = nullptr, *tiles = nullptr, *ntiles = nullptr, *inv = nullptr;
-	float *wgt = nullptr, *hid = nullptr, *out = nullptr;
+	float *wgt = nullptr, *hid = nullptr, *out = nullptr, *gate = nullptr, *shid = nullptr, *sout = nullptr;
 	uint8_t *a_hi = nullptr, *a_lo = nullptr, *hid_hi = nullptr, *hid_lo = nullptr;
 };
 
@@ -45,6 +52,16 @@ void moe_expect(SeqModel* m, const std::string& p, int E, int ff, bool gated) {
 		expect(m, pe + "up", {ff, m->width}, true);
 		expect(m, pe + "down", {m->width, ff}, true);
 	}
+}
+
+// tensors of a shared expert under prefix p ("<p>gate" ...); with a gate per token its row is "<p>sg"
+void moe_expect_shared(SeqModel* m, const std::string& p, MoeWeights* L, int ff, bool gate) {
+	L->shared_ff = ff;
+	L->shared_gate = gate;
+	expect(m, p + "gate", {ff, m->width}, true);
+	expect(m, p + "up", {ff, m->width}, true);
+	expect(m, p + "down", {m->width, ff}, true);
+	if (gate) expect(m, p + "sg", {1, m->width}, true);
 }
 
 // device layouts of the experts (one after the other, gate / up rows alternating) and the router; grows what the buffers must hold
@@ -59,7 +76,12 @@ int moe_upload(SeqModel* m, const std::string& p, bool gated, MoeWeights* L, Moe
 	L->up_rows = gated ? 2 * L->ff : L->ff;
 	XALM_TRY(upload_rows(m, up, m->width, gated, &L->w_up, &L->m_up));
 	XALM_TRY(upload_rows(m, dn, L->ff, false, &L->w_down, &L->m_down));
-	XALM_TRY(upload_rows(m, {tensor_or_null(m, p + "router")}, m->width, false, &L->w_router, nullptr));
+	XALM_TRY(upload_rows(m, {tensor_or_null(m, p + "router"), L->shared_gate ? tensor_or_null(m, p + "shared.sg") : nullptr}, m->width, false, &L->w_router, nullptr));
+	if (L->shared_ff) {
+		XALM_TRY(upload_rows(m, {tensor_or_null(m, p + "shared.gate"), tensor_or_null(m, p + "shared.up")}, m->width, true, &L->w_sup, &L->m_sup));
+		XALM_TRY(upload_rows(m, {tensor_or_null(m, p + "shared.down")}, L->shared_ff, false, &L->w_sdown, &L->m_sdown));
+		b->max_shared = std::max(b->max_shared, (size_t) L->shared_ff);
+	}
 	XALM_TRY(moe_prepare(m->width, L->E + L->identity, L->n_groups));
 	const size_t pairs = (size_t) m->chunk * L->top;
 	b->max_pairs = std::max(b->max_pairs, pairs);
@@ -74,6 +96,10 @@ inline int moe_tc_tiles(int pairs, int E) { return pairs / TC_TILE_ROWS + std::m
 // a mixture whose expert shapes the GEMM takes keeps fp16 tiles per expert for its long passes
 int moe_tc_register(SeqModel* m, MoeWeights* L, MoeBuffers* b) {
 	const int W = m->width;
+	if (L->shared_ff) {
+		XALM_TRY(tc_register(m, L->m_sup, &L->t_sup));
+		XALM_TRY(tc_register(m, L->m_sdown, &L->t_sdown));
+	}
 	if (!m->use_tc || !tune("seq_moe_tc") || !tc_shape_ok(L->up_rows, W, L->up_rows) || !tc_shape_ok(W, L->ff, W)) return XALM_OK;
 	L->t_up.resize((size_t) L->E);
 	L->t_down.resize((size_t) L->E);
@@ -108,6 +134,11 @@ int moe_alloc(SeqModel* m, MoeBuffers* b) {
 	XALM_TRY(dev_alloc(m, &b->ntiles, 1, true));
 	XALM_TRY(dev_alloc(m, &b->hid, b->max_hid));
 	XALM_TRY(dev_alloc(m, &b->out, b->max_pairs * W));
+	if (b->max_shared) {
+		XALM_TRY(dev_alloc(m, &b->gate, (size_t) m->chunk));
+		XALM_TRY(dev_alloc(m, &b->shid, (size_t) m->chunk * b->max_shared));
+		XALM_TRY(dev_alloc(m, &b->sout, (size_t) m->chunk * W));
+	}
 	if (b->a_bytes) {
 		XALM_TRY(dev_alloc(m, &b->inv, b->max_pairs, true));
 		XALM_TRY(dev_alloc(m, &b->a_hi, b->a_bytes, true));
@@ -123,15 +154,32 @@ int moe_alloc(SeqModel* m, MoeBuffers* b) {
 void moe_free(MoeWeights* L) {
 	for (TcWeight& t : L->t_up) tc_weight_free(&t);
 	for (TcWeight& t : L->t_down) tc_weight_free(&t);
+	tc_weight_free(&L->t_sup);
+	tc_weight_free(&L->t_sdown);
+}
+
+// The shared expert of n rows h on the main stream: b.sout (and, where the router gave one, its gate) becomes the join's base.
+int moe_shared(SeqModel* m, const MoeWeights& L, const MoeBuffers& b, const float* h, int n, RowsEpi act, MoeCombineArgs* ca, int* nl) {
+	const int W = m->width;
+	act.out = b.shid; act.ldo = L.shared_ff;
+	XALM_TRY(rows_product(m, h, W, L.w_sup, &L.t_sup, n, 2 * L.shared_ff, W, act, nl));
+	RowsEpi es;
+	es.kind = EPI_STORE; es.out = b.sout; es.ldo = W;
+	XALM_TRY(rows_product(m, b.shid, L.shared_ff, L.w_sdown, &L.t_sdown, n, W, L.shared_ff, es, nl));
+	ca->base = b.sout;
+	ca->base_w = L.shared_gate ? b.gate : nullptr;
+	return XALM_OK;
 }
 
 // Experts of n rows h (n, width) on the main stream.  `route` carries the scoring constants, `act` the epilogue of the first product (kind and
-// constants; out and ldo are set here).  Afterwards b.wgt and b.idx hold the choice and *ca names the expert rows for the caller's moe_combine.
+// constants; out and ldo are set here; a shared expert uses the same one).  Afterwards b.wgt and b.idx hold the choice and *ca names the expert
+// rows (and the shared expert's) for the caller's moe_combine.
 int moe_experts(SeqModel* m, const MoeWeights& L, const MoeBuffers& b, const float* h, int n, MoeRouteArgs route, RowsEpi act, MoeCombineArgs* ca, int* nl) {
 	cudaStream_t s = m->stream;
 	const int W = m->width, total = L.E + L.identity;
 	route.h = h; route.ldh = W; route.w = L.w_router; route.w_bf16 = m->w_bf16;
-	route.E = total; route.top = L.top; route.K = W; route.correction = L.correction;
+	route.E = total; route.top = L.top; route.K = W; route.correction = L.correction; route.bias = L.bias;
+	route.gate_out = L.shared_gate ? b.gate : nullptr;
 	route.n_groups = L.n_groups; route.keep_groups = L.keep_groups;
 	route.idx = b.idx; route.wgt = b.wgt; route.step = m->d_step;
 	XALM_TRY(launch_moe_router(route, n, s));
@@ -142,6 +190,7 @@ int moe_experts(SeqModel* m, const MoeWeights& L, const MoeBuffers& b, const flo
 		XALM_TRY(launch_moe_sort(so, s));
 		(*nl)++;
 	}
+	if (L.shared_ff) XALM_TRY(moe_shared(m, L, b, h, n, act, ca, nl));
 	act.ldo = L.ff;
 	if (on_tc) {
 		TcGroup up, dn;
