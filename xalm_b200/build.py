@@ -45,8 +45,9 @@ def _sources(d, exts):
 # linked units is kept beside the objects, and a later call that asks for more relinks.
 FAMILY_TUS = {"Llama": ["xalm_cuda.cu", "prefill.cu", "decode_mega.cu"], "Nabalix": ["nabalix.cu", "mix_ops.cu", "prefill.cu"],
               "Bolovik": ["bolovik.cu", "mix_ops.cu", "prefill.cu"], "Duletar": ["duletar.cu", "mix_ops.cu", "prefill.cu"],
-              "Kubolorn": ["kubolorn.cu", "mix_ops.cu", "prefill.cu"], "Mizerax": ["mizerax.cu", "mix_ops.cu", "prefill.cu"]}
-CUDA_TUS = ["abi.cu", "xalm_cuda.cu", "prefill.cu", "decode_mega.cu", "nabalix.cu", "bolovik.cu", "duletar.cu", "kubolorn.cu", "mizerax.cu", "mix_ops.cu"]
+              "Kubolorn": ["kubolorn.cu", "mix_ops.cu", "prefill.cu"], "Mizerax": ["mizerax.cu", "mix_ops.cu", "prefill.cu"],
+              "Pavitar": ["pavitar.cu", "mix_ops.cu", "prefill.cu"]}
+CUDA_TUS = ["abi.cu", "xalm_cuda.cu", "prefill.cu", "decode_mega.cu", "nabalix.cu", "bolovik.cu", "duletar.cu", "kubolorn.cu", "mizerax.cu", "pavitar.cu", "mix_ops.cu"]
 
 
 def _tus(families):
