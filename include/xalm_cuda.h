@@ -257,6 +257,25 @@ int xalm_cuda_moe_join(float* x_io, float* out_pairs, int* idx, float* wgt, cons
                        int E, int identity, int top, int ff, int w_bf16);
 int xalm_cuda_rows_add(float* out, const float* x, const float* w, const float* add, int T, int N, int K);
 
+/* Mechanisms of attention that forgets and of mixtures weighted among the chosen (fp32 host arrays in and out):
+ * chunked_attention: softmax attention where position i sees the j <= i with floor(j / chunk) = floor(i / chunk); k, v hold every position from 0 and are
+ *   laid into a ring of `ring` slots (position mod ring), as swa_attention does.
+ * row_norm_post: proj (T, H d + G d + G dv) = [q | k | v]; the whole q row and the whole k row over their root mean square (eps inside), times
+ *   q_norm_w (H d) / k_norm_w (G d) (NULL: 1), then the first 2 rot_half entries of every head turned by p * freq[i]: entry 2i with 2i + 1
+ *   (neighbours) or i with i + rot_half; k_out (ring, G d), v_out (ring, G dv) by row p % ring.  in_place: the queries overwrite the projection.
+ * latent_window: latent_attend without a rotated part, position i seeing 0 <= i - j < window, one gate value per head (T, H) or NULL; cache holds every
+ *   position's latent (pos0 + T, R) and is laid into a ring of `ring` rows.
+ * moe_chosen: logits z = h w_router^T + bias (NULL: 0); the `top` largest are chosen and weighted by the softmax over the chosen; x_io += sum wgt out +
+ *   base, experts as moe_join.  base_gated: w_router has a row E more, and base is multiplied by sigmoid of that row times h. */
+int xalm_cuda_chunked_attention(float* out, const float* q, const float* k, const float* v, int T, int pos0, int H, int G, int d, int dv, int chunk, float scale,
+                                int ring, int n_splits, int cache_bf16);
+int xalm_cuda_row_norm_post(float* q_out, float* k_out, float* v_out, const float* proj, int T, int pos0, int H, int G, int d, int dv, const float* q_norm_w,
+                            const float* k_norm_w, const float* freq, int rot_half, int neighbours, float eps, int ring, int in_place);
+int xalm_cuda_latent_window(float* out, const float* q, const float* cache, const float* gate, int T, int pos0, int H, int d, int dv, int R, const float* uk,
+                            const float* uv, float scale, int window, int ring, int n_splits, int cache_bf16);
+int xalm_cuda_moe_chosen(float* x_io, float* out_pairs, int* idx, float* wgt, const float* h, const float* w_router, const float* bias, const float* w_gate,
+                         const float* w_up, const float* w_down, const float* base, int base_gated, int T, int K, int E, int top, int ff, int w_bf16);
+
 /* Tensor parallel plumbing (no reference analogue; north star).  Rank 0 makes an id, the host side ships it to
  * the other ranks (torch.distributed / MPI / a file), every rank calls comm_init before finalize. */
 #define XALM_COMM_ID_BYTES 128

@@ -114,6 +114,10 @@ SYMBOLS = {
     "xalm_cuda_head_norm_post": (_i, [_vp] * 4 + [_i] * 6 + [_vp, _vp, C.c_float, _i, C.c_float, _i]),
     "xalm_cuda_biased_attention": (_i, [_vp] * 5 + [_i] * 6 + [C.c_float, _vp, _vp, _i, _i]),
     "xalm_cuda_moe_join": (_i, [_vp] * 14 + [_i] * 7),
+    "xalm_cuda_chunked_attention": (_i, [_vp] * 4 + [_i] * 7 + [C.c_float, _i, _i, _i]),
+    "xalm_cuda_row_norm_post": (_i, [_vp] * 4 + [_i] * 6 + [_vp] * 3 + [_i, _i, C.c_float, _i, _i]),
+    "xalm_cuda_latent_window": (_i, [_vp] * 4 + [_i] * 6 + [_vp, _vp, C.c_float, _i, _i, _i, _i]),
+    "xalm_cuda_moe_chosen": (_i, [_vp] * 11 + [_i] * 7),
     "xalm_cuda_rows_add": (_i, [_vp] * 4 + [_i] * 3),
 }
 PRECISION_BF16, PRECISION_F32 = 0, 1            # enum xalm_precision
@@ -570,3 +574,46 @@ def rows_add(x, w, add):
     out = np.empty((x.shape[0], w.shape[0]), dtype=np.float32)
     check(lib().xalm_cuda_rows_add(_p(out), _p(x), _p(w), _p(add), x.shape[0], w.shape[0], x.shape[1]))
     return out
+
+
+def chunked_attention(q, k, v, pos0, H, G, d, dv, chunk, scale, ring=None, n_splits=1, cache_bf16=False):
+    q, k, v = _f(q), _f(k), _f(v)
+    T = q.shape[0]
+    ring = pos0 + T if ring is None else ring
+    out = np.empty((T, H * dv), dtype=np.float32)
+    check(lib().xalm_cuda_chunked_attention(_p(out), _p(q), _p(k), _p(v), T, pos0, H, G, d, dv, chunk, scale, ring, n_splits, int(cache_bf16)))
+    return out
+
+
+def row_norm_post(proj, pos0, H, G, d, dv, q_norm_w, k_norm_w, freq=None, neighbours=True, eps=1e-5, ring=None, in_place=False):
+    """Returns (q rows, K cache, V cache) with the caches row by row."""
+    proj, q_norm_w, k_norm_w, freq = _f(proj), _f(q_norm_w), _f(k_norm_w), _f(freq)
+    T = proj.shape[0]
+    ring = pos0 + T if ring is None else ring
+    q, kc, vc = np.empty((T, H * d), dtype=np.float32), np.empty((ring, G * d), dtype=np.float32), np.empty((ring, G * dv), dtype=np.float32)
+    check(lib().xalm_cuda_row_norm_post(_p(q), _p(kc), _p(vc), _p(proj), T, pos0, H, G, d, dv, _pn(q_norm_w), _pn(k_norm_w), _pn(freq),
+                                        0 if freq is None else freq.shape[0], int(neighbours), eps, ring, int(in_place)))
+    return q, kc, vc
+
+
+def latent_window(q, cache, pos0, H, d, dv, R, uk, uv, scale, window, gate=None, ring=None, n_splits=0, cache_bf16=False):
+    q, cache, uk, uv, gate = _f(q), _f(cache), _f(uk), _f(uv), _f(gate)
+    T = q.shape[0]
+    assert cache.shape == (pos0 + T, R)
+    out = np.empty((T, H * dv), dtype=np.float32)
+    check(lib().xalm_cuda_latent_window(_p(out), _p(q), _p(cache), _pn(gate), T, pos0, H, d, dv, R, _p(uk), _p(uv), scale, window, ring or pos0 + T, n_splits,
+                                        int(cache_bf16)))
+    return out
+
+
+def moe_chosen(x, h, w_router, w_gate, w_up, w_down, top, bias=None, base=None, gate_row=None, w_bf16=False):
+    """Returns (x after the join, idx (T, top), wgt (T, top)); gate_row (K): base is multiplied by sigmoid(h . gate_row)."""
+    h, w_gate, w_up, w_down, bias, base = (_f(a) for a in (h, w_gate, w_up, w_down, bias, base))
+    w_router = _f(w_router if gate_row is None else np.concatenate([w_router, np.reshape(gate_row, (1, -1))]))
+    T, K = h.shape
+    E, ff = w_gate.shape[0], w_gate.shape[1]
+    idx, wgt, pairs = np.empty((T, top), dtype=np.int32), np.empty((T, top), dtype=np.float32), np.empty((T, top, K), dtype=np.float32)
+    xo = np.array(x, dtype=np.float32, copy=True)
+    check(lib().xalm_cuda_moe_chosen(_p(xo), _p(pairs), _p(idx), _p(wgt), _p(h), _p(w_router), _pn(bias), _p(w_gate), _p(w_up), _p(w_down), _pn(base),
+                                     int(gate_row is not None), T, K, E, top, ff, int(w_bf16)))
+    return xo, idx, wgt

@@ -62,11 +62,13 @@ uint16_t bf16_bits(float f) {
 
 static int swa_attention_op(float* out, const float* q, const float* gate, const float* k, const float* v, int T, int pos0, int H, int G, int d, int dv,
                             int window, int keep_first, float scale, float softcap, const float* r1, const float* r2, const float* talk, int ring, int n_splits,
-                            int cache_bf16, const float* sink = nullptr, float out_scale = 0.f, const float* slope = nullptr, bool gate_per_head = false) {
+                            int cache_bf16, const float* sink = nullptr, float out_scale = 0.f, const float* slope = nullptr, bool gate_per_head = false,
+                            int mask_chunk = 0) {
 	if (!out || !q || !k || !v || T <= 0 || pos0 < 0 || H <= 0 || G <= 0 || H % G || d <= 0 || dv <= 0 || window <= 0 || n_splits < 1 || keep_first < 0)
 		return set_error(XALM_ERR_INVALID, "swa_attention: bad argument");
 	const int n = pos0 + T;
-	const long long need = std::min<long long>(std::max(1, n - keep_first), (long long) window - 1 + T);
+	const int reach = mask_chunk > 0 ? std::min(window, mask_chunk) : window;
+	const long long need = std::min<long long>(std::max(1, n - keep_first), (long long) reach - 1 + T);
 	if (ring < need) return set_error(XALM_ERR_INVALID, "swa_attention: a ring of %d slots cannot hold %lld live positions", ring, need);
 	if (!r1 != !r2) return set_error(XALM_ERR_INVALID, "swa_attention: r1 and r2 come together");
 	const size_t smem = swa_smem_bytes(H, d, dv);
@@ -98,7 +100,8 @@ static int swa_attention_op(float* out, const float* q, const float* gate, const
 	a.slope = pool.put(slope, (size_t) H);
 	a.kc = pool.put(kr.data(), kr.size());
 	a.vc = pool.put(vr.data(), vr.size());
-	a.ring = ring; a.keep_first = keep_first; a.H = H; a.G = G; a.d = d; a.dv = dv; a.window = window; a.scale = scale; a.softcap = softcap;
+	a.ring = ring; a.keep_first = keep_first; a.H = H; a.G = G; a.d = d; a.dv = dv; a.window = window; a.mask_chunk = mask_chunk; a.scale = scale;
+	a.softcap = softcap;
 	a.r1 = pool.put(r1, (size_t) H); a.r2 = pool.put(r2, (size_t) H); a.talk = pool.put(talk, (size_t) H * H);
 	a.step = pool.put(&st, 1);
 	a.sink = pool.put(sink, (size_t) H); a.out_scale = out_scale;
@@ -344,6 +347,8 @@ int xalm_cuda_delta_rule(float* out, float* state, float* conv_state, const floa
 struct MoeExtras {
 	int identity = 0;
 	const float *correction = nullptr, *base = nullptr, *scale = nullptr, *other = nullptr, *other_scale = nullptr;
+	const float* bias = nullptr;   // (E + identity) of the logits
+	bool gate_row = false;         // w_router has one more row: base is multiplied by sigmoid(row . h)
 };
 static int moe_ffn_op(float* out_pairs, int* idx, float* wgt, const float* h, const float* w_router, const float* w_gate, const float* w_up,
                       const float* w_down, int T, int K, int E, int top, int ff, int n_groups, int keep_groups, int act, int w_bf16, int score_kind,
@@ -368,7 +373,9 @@ static int moe_ffn_op(float* out_pairs, int* idx, float* wgt, const float* h, co
 	const SeqStep* d_st = pool.put(&st, 1);
 	const int P = T * top, total = E + ex.identity, max_tiles = moe_max_tiles(P, E);
 	MoeRouteArgs ra = {};
-	ra.h = pool.put(h, (size_t) T * K); ra.ldh = K; ra.w = put_w(w_router, (size_t) total * K); ra.w_bf16 = w_bf16;
+	ra.h = pool.put(h, (size_t) T * K); ra.ldh = K; ra.w = put_w(w_router, (size_t) (total + (ex.gate_row ? 1 : 0)) * K); ra.w_bf16 = w_bf16;
+	ra.bias = pool.put(ex.bias, (size_t) total);
+	if (ex.gate_row) ra.gate_out = pool.raw<float>((size_t) T);
 	ra.correction = pool.put(ex.correction, (size_t) total);
 	ra.E = total; ra.top = top; ra.K = K; ra.n_groups = n_groups; ra.keep_groups = keep_groups;
 	ra.idx = pool.raw<int>((size_t) P); ra.wgt = pool.raw<float>((size_t) P); ra.step = d_st;
@@ -398,6 +405,7 @@ static int moe_ffn_op(float* out_pairs, int* idx, float* wgt, const float* h, co
 		MoeCombineArgs ca = {outp, K, top, K, ra.wgt, nullptr, d_x, d_x, d_st};
 		if (ex.identity) { ca.idx = ra.idx; ca.n_experts = E; ca.ident = ra.h; }
 		ca.base = pool.put(ex.base, (size_t) T * K);
+		ca.base_w = ra.gate_out;
 		ca.scale = pool.put(ex.scale, (size_t) K);
 		ca.other = pool.put(ex.other, (size_t) T * K);
 		ca.other_scale = pool.put(ex.other_scale, (size_t) K);
@@ -432,6 +440,15 @@ int xalm_cuda_moe_join(float* x_io, float* out_pairs, int* idx, float* wgt, cons
 	MoeExtras ex;
 	ex.identity = identity; ex.correction = correction; ex.base = base; ex.scale = scale; ex.other = other; ex.other_scale = other_scale;
 	return moe_ffn_op(out_pairs, idx, wgt, h, w_router, w_gate, w_up, w_down, T, K, E, top, ff, 0, 0, GLU_SILU, w_bf16, MOE_SCORE_SOFTMAX, MOE_GROUP_MAX, 0,
+	                  INFINITY, x_io, ex);
+}
+
+int xalm_cuda_moe_chosen(float* x_io, float* out_pairs, int* idx, float* wgt, const float* h, const float* w_router, const float* bias, const float* w_gate,
+                         const float* w_up, const float* w_down, const float* base, int base_gated, int T, int K, int E, int top, int ff, int w_bf16) {
+	if (!x_io || (base_gated && !base)) return set_error(XALM_ERR_INVALID, "moe_chosen: bad argument");
+	MoeExtras ex;
+	ex.bias = bias; ex.base = base; ex.gate_row = base_gated != 0;
+	return moe_ffn_op(out_pairs, idx, wgt, h, w_router, w_gate, w_up, w_down, T, K, E, top, ff, 0, 0, GLU_SILU, w_bf16, MOE_SCORE_CHOSEN, MOE_GROUP_MAX, 0,
 	                  INFINITY, x_io, ex);
 }
 
@@ -511,11 +528,13 @@ int xalm_cuda_latent_post(float* cq_out, float* cache_out, const float* proj, in
 	return XALM_OK;
 }
 
-int xalm_cuda_latent_attend(float* out, const float* q, const float* cache, const float* gate, int T, int pos0, int H, int d, int r, int dv, int R, int ld,
-                            const float* uk, const float* uv, const float* freq, float scale, int n_splits, int cache_bf16, int w_bf16) {
+static int latent_attend_op(float* out, const float* q, const float* cache, const float* gate, int T, int pos0, int H, int d, int r, int dv, int R, int ld,
+                            const float* uk, const float* uv, const float* freq, float scale, int n_splits, int cache_bf16, int w_bf16, int window = 0x7fffffff,
+                            int ring = 0, bool gate_per_head = false) {
 	if (!out || !q || !cache || !uk || !uv || T <= 0 || pos0 < 0 || H <= 0 || d <= 0 || r < 0 || r % 2 || dv <= 0 || R <= 0 || ld < R + r || n_splits < 0 || (r && !freq))
 		return set_error(XALM_ERR_INVALID, "latent_attend: bad argument");
-	const int n = pos0 + T, da = R + r;
+	const int n = pos0 + T, da = R + r, slots = ring > 0 ? ring : n;
+	if (window <= 0 || slots < std::min<long long>(n, (long long) window - 1 + T)) return set_error(XALM_ERR_INVALID, "latent_attend: %d slots for a window of %d", slots, window);
 	if (!swa_pick_tq(H, 1, da, R, T) && swa_smem_bytes(H, da, R) > 200 * 1024) return set_error(XALM_ERR_UNSUPPORTED, "latent_attend: heads need too much shared memory");
 	Pool pool;
 	auto put_w = [&](const float* src, size_t cnt) -> void* {
@@ -528,16 +547,18 @@ int xalm_cuda_latent_attend(float* out, const float* q, const float* cache, cons
 	for (int h = 0; h < H; h++)
 		for (int i = 0; i < d; i++)
 			for (int j = 0; j < R; j++) ukT[((size_t) h * R + j) * d + i] = uk[((size_t) h * d + i) * R + j];
+	std::vector<float> rows((size_t) slots * ld, 0.f); // as the cache manager leaves them: position p in slot p mod ring
+	for (int p = 0; p < n; p++) memcpy(&rows[(size_t) (p % slots) * ld], cache + (size_t) p * ld, (size_t) ld * 4);
 	void* d_cache;
 	if (cache_bf16) {
-		std::vector<uint16_t> cb((size_t) n * ld);
-		for (size_t i = 0; i < cb.size(); i++) cb[i] = bf16_bits(cache[i]);
+		std::vector<uint16_t> cb(rows.size());
+		for (size_t i = 0; i < cb.size(); i++) cb[i] = bf16_bits(rows[i]);
 		d_cache = pool.put(cb.data(), cb.size());
-	} else d_cache = pool.put(cache, (size_t) n * ld);
+	} else d_cache = pool.put(rows.data(), rows.size());
 	const SeqStep st = {pos0, T};
 	const SeqStep* d_st = pool.put(&st, 1);
 	const float* d_q = pool.put(q, (size_t) T * H * (d + r));
-	const float* d_gate = pool.put(gate, (size_t) T * H * dv);
+	const float* d_gate = pool.put(gate, (size_t) T * H * (gate_per_head ? 1 : dv));
 	const float* d_freq = pool.put(freq, (size_t) r / 2);
 	void *d_ukT = put_w(ukT.data(), ukT.size()), *d_uv = put_w(uv, (size_t) H * dv * R);
 	float *qabs = pool.raw<float>((size_t) T * H * da), *olat = pool.raw<float>((size_t) T * H * R), *d_out = pool.raw<float>((size_t) T * H * dv);
@@ -555,8 +576,9 @@ int xalm_cuda_latent_attend(float* out, const float* q, const float* cache, cons
 	}
 	SwaArgs sa = {};
 	sa.q = qabs; sa.ldq = H * da;
-	sa.kc = d_cache; sa.vc = d_cache; sa.ldk = ld; sa.ldv = ld; sa.ring = n;
-	sa.H = H; sa.G = 1; sa.d = da; sa.dv = R; sa.window = 0x7fffffff; sa.scale = scale;
+	sa.kc = d_cache; sa.vc = d_cache; sa.ldk = ld; sa.ldv = ld; sa.ring = slots;
+	sa.H = H; sa.G = 1; sa.d = da; sa.dv = R; sa.window = window; sa.scale = scale;
+	if (gate_per_head) { sa.gate = d_gate; sa.ldg = H; sa.gate_per_head = 1; }
 	sa.step = d_st; sa.out = olat;
 	sa.n_splits = n_splits;
 	const int cap = std::max(4 * 64, 4 * T);
@@ -568,11 +590,20 @@ int xalm_cuda_latent_attend(float* out, const float* q, const float* cache, cons
 	XALM_TRY(launch_swa(sa, T, cache_bf16 == 0, nullptr));
 	RowsEpi ev;
 	ev.kind = EPI_STORE; ev.out = d_out; ev.ldo = H * dv; ev.batch_a = R; ev.batch_w = (size_t) dv * R; ev.batch_o = dv;
-	if (gate) { ev.mul = d_gate; ev.ldm = H * dv; ev.mul_act = ACT_SIGMOID; }
+	if (gate && !gate_per_head) { ev.mul = d_gate; ev.ldm = H * dv; ev.mul_act = ACT_SIGMOID; }
 	XALM_TRY(launch_rows(olat, H * R, d_uv, w_bf16 != 0, T, dv, R, ev, nullptr, H));
 	XALM_TRY(finish("latent_attend"));
 	XALM_CUDA_CHECK(cudaMemcpy(out, d_out, (size_t) T * H * dv * 4, cudaMemcpyDeviceToHost));
 	return XALM_OK;
+}
+
+int xalm_cuda_latent_attend(float* out, const float* q, const float* cache, const float* gate, int T, int pos0, int H, int d, int r, int dv, int R, int ld,
+                            const float* uk, const float* uv, const float* freq, float scale, int n_splits, int cache_bf16, int w_bf16) {
+	return latent_attend_op(out, q, cache, gate, T, pos0, H, d, r, dv, R, ld, uk, uv, freq, scale, n_splits, cache_bf16, w_bf16);
+}
+int xalm_cuda_latent_window(float* out, const float* q, const float* cache, const float* gate, int T, int pos0, int H, int d, int dv, int R, const float* uk,
+                            const float* uv, float scale, int window, int ring, int n_splits, int cache_bf16) {
+	return latent_attend_op(out, q, cache, gate, T, pos0, H, d, 0, dv, R, R, uk, uv, nullptr, scale, n_splits, cache_bf16, 0, window, ring, gate != nullptr);
 }
 
 int xalm_cuda_rows_act(float* out, const float* x, const float* w, int T, int N, int K, int act, float cap, const float* mul, int mul_act, int w_bf16) {
@@ -609,6 +640,40 @@ int xalm_cuda_biased_attention(float* out, const float* q, const float* gate, co
                                float scale, const float* slope, const float* sink, int n_splits, int cache_bf16) {
 	return swa_attention_op(out, q, gate, k, v, T, pos0, H, G, d, dv, 0x7fffffff, 0, scale, 0.f, nullptr, nullptr, nullptr, pos0 + T, n_splits, cache_bf16, sink, 0.f,
 	                        slope, true);
+}
+
+int xalm_cuda_chunked_attention(float* out, const float* q, const float* k, const float* v, int T, int pos0, int H, int G, int d, int dv, int chunk, float scale,
+                                int ring, int n_splits, int cache_bf16) {
+	if (chunk <= 0) return set_error(XALM_ERR_INVALID, "chunked_attention: chunks of %d", chunk);
+	return swa_attention_op(out, q, nullptr, k, v, T, pos0, H, G, d, dv, 0x7fffffff, 0, scale, 0.f, nullptr, nullptr, nullptr, ring, n_splits, cache_bf16, nullptr, 0.f,
+	                        nullptr, false, chunk);
+}
+
+int xalm_cuda_row_norm_post(float* q_out, float* k_out, float* v_out, const float* proj, int T, int pos0, int H, int G, int d, int dv, const float* q_norm_w,
+                            const float* k_norm_w, const float* freq, int rot_half, int neighbours, float eps, int ring, int in_place) {
+	if (!q_out || !k_out || !v_out || !proj || T <= 0 || pos0 < 0 || H <= 0 || G <= 0 || d <= 0 || dv <= 0 || ring <= 0 || rot_half < 0 || (rot_half && !freq))
+		return set_error(XALM_ERR_INVALID, "row_norm_post: bad argument");
+	Pool pool;
+	const int ld = H * d + G * d + G * dv;
+	const SeqStep st = {pos0, T};
+	QkvPostArgs a = {};
+	a.proj = pool.put(proj, (size_t) T * ld); a.ld = ld; a.k_off = H * d; a.v_off = H * d + G * d;
+	a.H = H; a.G = G; a.d = d; a.dv = dv;
+	a.freq = rot_half ? pool.put(freq, (size_t) rot_half) : nullptr; a.rot_half = rot_half; a.rot_neighbours = neighbours;
+	a.norm_rows = 1; a.eps = eps;
+	a.q_norm_w = pool.put(q_norm_w, (size_t) H * d); a.k_norm_w = pool.put(k_norm_w, (size_t) G * d);
+	if (!in_place) { a.q_out = pool.raw<float>((size_t) T * H * d); a.ldq_out = H * d; }
+	float *kc = pool.raw<float>((size_t) ring * G * d), *vc = pool.raw<float>((size_t) ring * G * dv);
+	a.kc = kc; a.vc = vc; a.cache_f32 = 1; a.ring = ring;
+	a.step = pool.put(&st, 1);
+	if (!a.proj || !kc || !vc || !a.step || (!in_place && !a.q_out)) return set_error(XALM_ERR_CUDA, "row_norm_post: device allocation failed");
+	XALM_TRY(launch_qkv_post(a, T, nullptr));
+	XALM_TRY(finish("row_norm_post"));
+	if (in_place) XALM_CUDA_CHECK(cudaMemcpy2D(q_out, (size_t) H * d * 4, a.proj, (size_t) ld * 4, (size_t) H * d * 4, T, cudaMemcpyDeviceToHost));
+	else XALM_CUDA_CHECK(cudaMemcpy(q_out, a.q_out, (size_t) T * H * d * 4, cudaMemcpyDeviceToHost));
+	XALM_CUDA_CHECK(cudaMemcpy(k_out, kc, (size_t) ring * G * d * 4, cudaMemcpyDeviceToHost));
+	XALM_CUDA_CHECK(cudaMemcpy(v_out, vc, (size_t) ring * G * dv * 4, cudaMemcpyDeviceToHost));
+	return XALM_OK;
 }
 
 int xalm_cuda_layer_norm(float* out, const float* x, const float* w, const float* b, int T, int W, float eps) {
