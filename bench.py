@@ -623,6 +623,50 @@ def build_mizerax(z: dict, seed: int, max_tokens: int, stream):
     return m
 
 
+def pavitar_config(z: dict) -> dict:
+    """Layers alternate: latent attention in the size's window (latents as the Duletar model's, heads of 128, a gate per head), then grouped
+    attention in chunks of as many positions (rotation on half of each head); every layer has a mixture of 16 gated experts of ff / 4 of which 4
+    are chosen and a gated shared expert of ff / 4.  The second half of the layers is one pass over a loop, so that as many layers run as in the
+    other families' models of the size and all read weights of their own."""
+    W, d = z["width"], z["head_dim"]
+    lat = {"heads": z["heads"], "dim": d, "vdim": d, "kv_rank": min(512, max(256, W // 4)), "q_rank": 3 * W // 8, "scale": d ** -0.5, "mask": {"size": z["window"]}}
+    att = {"heads": z["heads"], "kv_heads": z["kv_heads"], "dim": d, "vdim": d, "scale": d ** -0.5, "mask": {"size": z["window"]},
+           "rot": {"base": 10000.0, "dims": d // 2}}
+    moe = {"kind": "moe", "expert": {"ff": z["ff"] // 4}, "router": {"experts": 16, "top": 4}, "shared": {"ff": z["ff"] // 4}}
+    pair = [{"type": "latent_attention", "mixer": lat, "mlp": moe}, {"type": "attention", "mixer": att, "mlp": moe}]
+    return {"architecture": "Pavitar", "vocab": z["vocab"], "width": W, "norm": {"eps": 1e-6}, "logit_softcap": 30.0,
+            "layers": (pair * z["layers"])[:z["layers"]], "loop": {"start": z["layers"] // 2, "stop": z["layers"], "times": 1}}
+
+
+def build_pavitar(z: dict, seed: int, max_tokens: int, stream):
+    """Random bf16 weights, uploaded tensor by tensor as the backend names them."""
+    import ctypes as C
+    import json
+    from xalm_b200 import capi, safetensors_io as ST, types as T
+    from xalm_b200.model import Model
+    m = Model._from_json_text(json.dumps(pavitar_config(z)), {})
+    L = capi.lib()
+    h = C.c_void_p()
+    capi.check(L.xalm_cuda_create_json(m.config["json"].encode(), 0, max_tokens, capi.PRECISION_BF16, C.byref(h)))
+    m._h = h
+    capi.check(L.xalm_cuda_set_stream(h, C.c_void_p(stream)))
+    rng = np.random.default_rng(seed)
+    for name, shape in m.expected_tensors().items():
+        leaf = name.split(".")[-1]
+        if name == "embed":
+            a = rng.standard_normal(shape, dtype=np.float32)
+        elif len(shape) == 2:
+            a = rng.standard_normal(shape, dtype=np.float32) * np.float32((2.0 if leaf == "router" else 1.0) / np.sqrt(shape[1]))
+        elif leaf in ("norm1", "norm2", "b") or name == "final.norm":
+            a = 0.1 * rng.standard_normal(shape, dtype=np.float32)
+        else:
+            a = 1.0 + 0.1 * rng.standard_normal(shape, dtype=np.float32)
+        m.upload(name, T.BF16, shape, ST.f32_to_bf16_bits(a).view(np.uint8).reshape(-1))
+    capi.check(L.xalm_cuda_finalize(h))
+    m.config["vocab_size"] = z["vocab"]
+    return m
+
+
 def run_family_workload(args, fams=("nabalix", "llama")):
     """Prefill and one-token-step throughput of config.json families beside one another and beside the Llama family at equal layer sizes
     (bf16 weights, random), device-timed with CUDA events on the launching stream.  One JSON line; `value` is the first family's decode rate
@@ -648,7 +692,7 @@ def run_family_workload(args, fams=("nabalix", "llama")):
                 if fam != "llama":
                     capi.tune("seq_chunk", args.seq_chunk)  # positions per pass of a prompt (the Llama arm takes the prompt in one pass)
                     m = {"nabalix": build_nabalix, "bolovik": build_bolovik, "duletar": build_duletar, "kubolorn": build_kubolorn,
-                         "mizerax": build_mizerax}[fam](z, args.seed, ctx, stream.cuda_stream)
+                         "mizerax": build_mizerax, "pavitar": build_pavitar}[fam](z, args.seed, ctx, stream.cuda_stream)
                 else:
                     m, _ = build_model_streaming(llama_full, llama_cfg, T.BF16, args.seed, False, stream=stream.cuda_stream)
                     capi.tune("prefill_split", 1)        # plain fp16 operands, the counterpart of the one-plane path
@@ -709,15 +753,17 @@ def main():
     ap.add_argument("--past-window", action="store_true",
                     help="also time steps at positions >= ctx: the KV ring is full (kv_len = ctx), 2 attention sinks active (infer.cpp:608-613)")
     ap.add_argument("--no-prefill", action="store_true", help="skip the perplexity-mode summary appended to the decode line at N=1")
-    ap.add_argument("--workload", default="decode", choices=["decode", "perplexity", "families", "bolovik", "duletar", "kubolorn", "mizerax"],
+    ap.add_argument("--workload", default="decode", choices=["decode", "perplexity", "families", "bolovik", "duletar", "kubolorn", "mizerax", "pavitar"],
                     help="decode = BASELINE config[1] (the headline metric); perplexity = config[2]: batched prefill of a 4k-token input; "
                          "families = prefill and one-token-step throughput of the Nabalix family beside the Llama family at equal layer sizes; "
                          "bolovik = the same for the Bolovik family beside the Nabalix and Llama families; "
                          "duletar = the same for the Duletar family beside the Bolovik family; "
                          "kubolorn = the same for the Kubolorn family beside the Bolovik family; "
-                         "mizerax = the same for the Mizerax family beside the Bolovik and Kubolorn families")
-    ap.add_argument("--arms", default="", help="bolovik / duletar / kubolorn / mizerax workloads: which families run, the first one is the headline "
-                                               "(default bolovik,nabalix,llama / duletar,bolovik / kubolorn,bolovik / mizerax,bolovik,kubolorn)")
+                         "mizerax = the same for the Mizerax family beside the Bolovik and Kubolorn families; "
+                         "pavitar = the same for the Pavitar family beside the Duletar, Bolovik and Mizerax families")
+    ap.add_argument("--arms", default="", help="bolovik / duletar / kubolorn / mizerax / pavitar workloads: which families run, the first one is the headline "
+                                               "(default bolovik,nabalix,llama / duletar,bolovik / kubolorn,bolovik / mizerax,bolovik,kubolorn / "
+                                               "pavitar,duletar,bolovik,mizerax)")
     ap.add_argument("--seq-chunk", type=int, default=1024, help="families workload: positions per pass of a Nabalix prompt")
     ap.add_argument("--sizes", default="w1024,w2048,w4096", help="families workload: which of " + ",".join(FAMILY_SIZES))
     ap.add_argument("--tokens", type=int, default=4096, help="perplexity workload: tokens per step")
@@ -728,10 +774,10 @@ def main():
     if args.workload == "perplexity":
         run_perplexity_workload(args)
         return
-    if args.workload in ("families", "bolovik", "duletar", "kubolorn", "mizerax"):
+    if args.workload in ("families", "bolovik", "duletar", "kubolorn", "mizerax", "pavitar"):
         if not args.arms:
             args.arms = {"duletar": "duletar,bolovik", "kubolorn": "kubolorn,bolovik",
-                         "mizerax": "mizerax,bolovik,kubolorn"}.get(args.workload, "bolovik,nabalix,llama")
+                         "mizerax": "mizerax,bolovik,kubolorn", "pavitar": "pavitar,duletar,bolovik,mizerax"}.get(args.workload, "bolovik,nabalix,llama")
         if args.steps == 256:
             args.steps = 64
         if args.tokens == 4096:

@@ -308,6 +308,21 @@ def test_tensor_core_passes_match_the_fp32_kernels():
     rows_within(outputs[2], outputs[0], 1e-2)
 
 
+def test_side_branch_off_gives_the_same_rows(case):
+    """The router beside the shared expert on two streams or before it on one: the same kernels, the same bits."""
+    cfg, W, tokens, _, _ = case
+    rows = []
+    for overlap in (1, 0):
+        capi.tune("seq_overlap", overlap)
+        try:
+            m = on_gpu(cfg, W, capi.PRECISION_F32, chunk=16)
+            rows.append(step_all(m, tokens, [20, 1, 1, 9]))
+            m.close()
+        finally:
+            capi.tune("seq_overlap", 1)
+    assert np.array_equal(rows[0], rows[1])
+
+
 def test_graph_and_eager_steps_agree(case):
     cfg, W, tokens, _, _ = case
     rows = []

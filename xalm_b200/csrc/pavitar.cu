@@ -21,7 +21,8 @@
 //     latent:     rows product [dq | dkv | g] -> latent_attention (absorbed form, window ring, head gate fused)
 //     attention:  rows product [q | k | v] -> qkv_rows_post (row norms, rotation, cache rows) -> swa_attn / swa_tile with the chunk mask
 //     rows product [o] with the residual add fused
-//     norm -> router (with the shared expert's gate) -> shared expert -> experts -> moe_combine (+ gated shared row + residual)
+//     norm -> router (with the shared expert's gate) and sort on the side stream beside the shared expert on the main one -> experts ->
+//     moe_combine (+ gated shared row + residual)
 //
 // Cache / state manager: per layer RUN a ring of mask.size - 1 + seq_chunk rows (at most max_tokens): latents, or normed and turned keys and
 // values.  Rows need no clearing: a sequence only reads positions it wrote.
@@ -250,7 +251,7 @@ int enqueue_pass(SeqModel* sm, int n, int want, int* nl) {
 			eg.kind = EPI_GLU; eg.glu_act = GLU_SILU;
 			MoeCombineArgs ca = {};
 			ca.x_in = x; ca.x_out = x;
-			XALM_TRY(moe_experts(m, L.moe, m->moe, m->hn, n, ra, eg, &ca, nl));
+			XALM_TRY(moe_experts(m, L.moe, m->moe, m->hn, n, ra, eg, &ca, nl, tune("seq_overlap") != 0));
 			XALM_TRY(launch_moe_combine(ca, n, s));
 			*nl += 2;
 		}

@@ -173,24 +173,30 @@ int moe_shared(SeqModel* m, const MoeWeights& L, const MoeBuffers& b, const floa
 
 // Experts of n rows h (n, width) on the main stream.  `route` carries the scoring constants, `act` the epilogue of the first product (kind and
 // constants; out and ldo are set here; a shared expert uses the same one).  Afterwards b.wgt and b.idx hold the choice and *ca names the expert
-// rows (and the shared expert's) for the caller's moe_combine.
-int moe_experts(SeqModel* m, const MoeWeights& L, const MoeBuffers& b, const float* h, int n, MoeRouteArgs route, RowsEpi act, MoeCombineArgs* ca, int* nl) {
+// rows (and the shared expert's) for the caller's moe_combine.  side_free: the side stream has nothing else to do, and the router (one CTA per token)
+// and the sort run there beside the shared expert's products.
+int moe_experts(SeqModel* m, const MoeWeights& L, const MoeBuffers& b, const float* h, int n, MoeRouteArgs route, RowsEpi act, MoeCombineArgs* ca, int* nl,
+                bool side_free = false) {
 	cudaStream_t s = m->stream;
+	const Fork fk = {m, side_free && L.shared_ff > 0};
 	const int W = m->width, total = L.E + L.identity;
 	route.h = h; route.ldh = W; route.w = L.w_router; route.w_bf16 = m->w_bf16;
 	route.E = total; route.top = L.top; route.K = W; route.correction = L.correction; route.bias = L.bias;
 	route.gate_out = L.shared_gate ? b.gate : nullptr;
 	route.n_groups = L.n_groups; route.keep_groups = L.keep_groups;
 	route.idx = b.idx; route.wgt = b.wgt; route.step = m->d_step;
-	XALM_TRY(launch_moe_router(route, n, s));
+	XALM_TRY(fk.open());
+	XALM_TRY(launch_moe_router(route, n, fk.side()));
 	(*nl)++;
 	const bool on_tc = L.on_tc(m, n);
 	if (on_tc || n * L.top > MOE_MATVEC_PAIRS) { // steps of a few tokens need no tile list
 		MoeSortArgs so = {b.idx, L.top, total, m->d_step, b.sorted, b.tiles, b.ntiles, nullptr, b.inv, L.E, on_tc ? TC_TILE_ROWS : 0};
-		XALM_TRY(launch_moe_sort(so, s));
+		XALM_TRY(launch_moe_sort(so, fk.side()));
 		(*nl)++;
 	}
+	XALM_TRY(fk.mark());
 	if (L.shared_ff) XALM_TRY(moe_shared(m, L, b, h, n, act, ca, nl));
+	XALM_TRY(fk.join());
 	act.ldo = L.ff;
 	if (on_tc) {
 		TcGroup up, dn;
